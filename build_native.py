@@ -51,6 +51,8 @@ COMPONENTS = {
     "serve-tupidra": _SERVE_COMMON + ["norm/scalar_rmsnorm.cu", "norm/sandwich_norm.cu", "norm/canon_norm.cu",
                                       "attention/latent_attention.cu", "attention/latent_attention_t5.cu",
                                       "attention/softcap_window_attention.cu", "recurrent/selective_scan.cu"],
+    "serve-zokepel": _SERVE_COMMON + ["norm/sandwich_norm.cu", "norm/dual_norm.cu", "attention/softcap_window_attention.cu",
+                                      "recurrent/gla.cu", "recurrent/matrix_state.cu"],
     "all": None,
 }
 

@@ -89,6 +89,17 @@ __global__ void __launch_bounds__(256) relu_squared_kernel(const T* __restrict__
   }
 }
 
+// in place over a [rows, F] view with row stride ld
+template <typename T>
+__global__ void __launch_bounds__(256) tanh_kernel(T* __restrict__ z, long long ld, int rows, int F) {
+  const long long n = static_cast<long long>(rows) * F;
+  for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < n;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    T* p = z + i / F * ld + i % F;
+    *p = from_f32<T>(tanhf(to_f32(*p)));
+  }
+}
+
 static inline int grid_for(long long n) {
   long long b = (n + 255) / 256;
   if (b > kNumSMs * 16) b = kNumSMs * 16;
@@ -147,5 +158,14 @@ LLMCTL_API int llmctl_relu_squared(const void* z, void* out, int is_fp32, long l
   LLMCTL_BEGIN();
   if (n == 0) return 0;
   LLMCTL_DISPATCH_DTYPE(is_fp32, T, (relu_squared_kernel<T><<<grid_for(n), 256, 0, (cudaStream_t)stream>>>((const T*)z, (T*)out, n)));
+  LLMCTL_RETURN_LAST();
+}
+
+// z <- tanh(z) in place, [rows, F] with row stride ld
+LLMCTL_API int llmctl_tanh(void* z, long long ld, int is_fp32, int rows, int F, void* stream) {
+  LLMCTL_BEGIN();
+  LLMCTL_REQUIRE(ld >= F);
+  if (rows == 0 || F == 0) return 0;
+  LLMCTL_DISPATCH_DTYPE(is_fp32, T, (tanh_kernel<T><<<grid_for(static_cast<long long>(rows) * F), 256, 0, (cudaStream_t)stream>>>((T*)z, ld, rows, F)));
   LLMCTL_RETURN_LAST();
 }

@@ -9,12 +9,17 @@
 //     o_i  = sum_j p_ij v_j,  times sigmoid(gate[i, h, :]) where a gate is given
 //
 // slopes and sinks are fp32 arrays of H numbers (null: no bias / no sink); a sink has no value, so it only enlarges the
-// denominator.  Cache of a layer: [pages, bs, G*d + G*e]; a token's row holds the keys of all key/value heads and then
+// denominator.  Instead of (or beside) the linear bias a table of biases by distance may be given, fp32 [H, L]:
+//
+//     s_ij <- s_ij + table[h, min(i - j, L - 1)]              (not multiplied by scale; a learned bucketed bias is such a table)
+//
+// The linear bias and the table apply after the cap.  Cache of a layer: [pages, bs, G*d + G*e]; a token's row holds the keys of all key/value heads and then
 // their values.
 //
 //   llmctl_window_kv_append : per token, from a packed projection [q | k | v | ...]: fp32 biases (optional), unit-RMS
-//       norm of every value head (optional: v / sqrt(mean(v^2) + eps), no weight); q leaves in fp32, k and v go to the
-//       token's cache row.
+//       norm of every value head (optional: v / sqrt(mean(v^2) + eps), no weight), unit-RMS norm of every query and key
+//       head (optional, no weight), query temperature (optional: q *= 1 + coef ln(floor((p + 1) / every) + 1) at position p);
+//       q leaves in fp32, k and v go to the token's cache row.
 //   llmctl_softcap_window_attention : key tiles run over the kept first tokens and then over the window of the tile's
 //       queries only; everything else is never read.  FMA kernel (fp32 caches, any sizes): a CTA owns up to 16
 //       consecutive tokens x HB heads of one key/value head as <= 32 softmax rows, a warp owns four rows through all
@@ -37,20 +42,39 @@ namespace llmctl {
 template <typename T>
 __global__ void __launch_bounds__(256)
 window_kv_append_kernel(const T* __restrict__ proj, long long ld, const float* __restrict__ bias, int H, int G, int d, int e,
-                        int value_norm, float eps, const long long* __restrict__ slots, float* __restrict__ q_out,
-                        T* __restrict__ cache) {
+                        int value_norm, int qk_norm, float temp_coef, double temp_every, const int* __restrict__ positions, float eps,
+                        const long long* __restrict__ slots, float* __restrict__ q_out, T* __restrict__ cache) {
   const long long t = blockIdx.x;
   const int Nq = H * d, Nk = G * d, Wc = Nk + G * e;
   const T* row = proj + t * ld;
   const long long slot = slots[t];
   T* crow = slot >= 0 ? cache + slot * Wc : nullptr;
-  for (int c = threadIdx.x; c < Nq + Nk; c += blockDim.x) {
-    const float v = to_f32(row[c]) + (bias ? bias[c] : 0.f);
-    if (c < Nq) q_out[t * Nq + c] = v;
-    else if (crow) crow[c - Nq] = from_f32<T>(v);
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = blockDim.x >> 5;
+  float temp = 1.f;
+  if (positions) temp = 1.f + temp_coef * logf(static_cast<float>(floor((static_cast<double>(positions[t]) + 1.0) / temp_every)) + 1.f);
+  if (qk_norm) {
+    for (int hd = warp; hd < H + G; hd += nwarp) {            // query heads, then key heads
+      const int base = hd * d;
+      float ss = 0.f;
+      for (int c = lane; c < d; c += 32) {
+        const float v = to_f32(row[base + c]) + (bias ? bias[base + c] : 0.f);
+        ss += v * v;
+      }
+      const float f = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(d) + eps);
+      for (int c = lane; c < d; c += 32) {
+        const float v = (to_f32(row[base + c]) + (bias ? bias[base + c] : 0.f)) * f;
+        if (hd < H) q_out[t * Nq + base + c] = v * temp;
+        else if (crow) crow[base - Nq + c] = from_f32<T>(v);
+      }
+    }
+  } else {
+    for (int c = threadIdx.x; c < Nq + Nk; c += blockDim.x) {
+      const float v = to_f32(row[c]) + (bias ? bias[c] : 0.f);
+      if (c < Nq) q_out[t * Nq + c] = v * temp;
+      else if (crow) crow[c - Nq] = from_f32<T>(v);
+    }
   }
   if (!crow) return;
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = blockDim.x >> 5;
   for (int g = warp; g < G; g += nwarp) {
     const int base = Nq + Nk + g * e;
     float ss = 0.f;
@@ -83,6 +107,8 @@ struct SoftcapAttnParams {
   long long gate_ld;
   const float* slopes;       // [H] or null
   const float* sinks;        // [H] or null
+  const float* table;        // [H, table_len] bias by distance, or null
+  int table_len;
   float scale, cap;
   int window, keep_first;
   int H, G, d, e, bs;
@@ -142,6 +168,7 @@ softcap_attention_kernel(const SoftcapAttnParams p) {
   }
 
   float m[4], l[4], acc[4][NC], slope[4];
+  const float* tab[4];
   int qpos[4];
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
@@ -149,6 +176,7 @@ softcap_attention_kernel(const SoftcapAttnParams p) {
     const int h = h0 + (r < nrows ? r % HB : 0);
     qpos[i] = r < nrows ? p_first + r / HB : -1;
     slope[i] = p.slopes ? p.slopes[h] : 0.f;
+    tab[i] = p.table ? p.table + static_cast<long long>(h) * p.table_len : nullptr;
     const bool sink = p.sinks != nullptr && split == 0;
     m[i] = sink ? p.sinks[h] : -INFINITY;
     l[i] = sink ? 1.f : 0.f;
@@ -213,6 +241,7 @@ softcap_attention_kernel(const SoftcapAttnParams p) {
           if (seen) {
             sv = p.cap > 0.f ? p.cap * tanhf(s[i] / p.cap) : s[i];
             sv -= slope[i] * static_cast<float>(qpos[i] - j);
+            if (tab[i]) sv += tab[i][min(qpos[i] - j, p.table_len - 1)];
           }
           const float mn = fmaxf(m[i], warp_max(sv));
           float pw = 0.f, corr = 1.f;
@@ -428,6 +457,10 @@ softcap_attention_mma_kernel(const SoftcapAttnParams p, int decode) {
   const int qpos_hi = r_hi < nvalid ? (decode ? p_first : p_first + r_hi) : -1;
   const int head_lo = decode ? h0 + min(r_lo, nvalid - 1) : h0, head_hi = decode ? h0 + min(r_hi, nvalid - 1) : h0;
   const float slope_lo = p.slopes ? p.slopes[head_lo] : 0.f, slope_hi = p.slopes ? p.slopes[head_hi] : 0.f;
+  const float* tab_lo = p.table ? p.table + static_cast<long long>(head_lo) * p.table_len : nullptr;
+  const float* tab_hi = p.table ? p.table + static_cast<long long>(head_hi) * p.table_len : nullptr;
+  const int far = p.table_len - 1;       // every distance from here on has the table's last bias
+  const float far_lo = tab_lo ? tab_lo[far] : 0.f, far_hi = tab_hi ? tab_hi[far] : 0.f;
   const bool warp_active = warp * 16 < nvalid;
   // keys this warp's rows can see: the kept first tokens and [warp_wb, warp_last]
   const int warp_first = decode ? p_first : p_first + warp * 16;
@@ -483,6 +516,7 @@ softcap_attention_mma_kernel(const SoftcapAttnParams p, int decode) {
         mma_bf16_16816(S[nt], al, b);
       }
     }
+    const bool near_tile = warp_first - (k0 + kSwKT - 1) < far;
     // cap, distance bias, mask; running maximum and sum per row (scores in units of ln 2 from here on)
     float mx_lo = -INFINITY, mx_hi = -INFINITY;
 #pragma unroll
@@ -496,8 +530,19 @@ softcap_attention_mma_kernel(const SoftcapAttnParams p, int decode) {
           s_lo = p.cap * sw_tanh(s_lo / p.cap);
           s_hi = p.cap * sw_tanh(s_hi / p.cap);
         }
-        s_lo = (s_lo - slope_lo * static_cast<float>(qpos_lo - key)) * kSwLog2e;
-        s_hi = (s_hi - slope_hi * static_cast<float>(qpos_hi - key)) * kSwLog2e;
+        s_lo -= slope_lo * static_cast<float>(qpos_lo - key);
+        s_hi -= slope_hi * static_cast<float>(qpos_hi - key);
+        if (tab_lo) {
+          if (near_tile) {               // distances outside 0 .. far belong to masked or far keys
+            s_lo += tab_lo[min(max(qpos_lo - key, 0), far)];
+            s_hi += tab_hi[min(max(qpos_hi - key, 0), far)];
+          } else {
+            s_lo += far_lo;
+            s_hi += far_hi;
+          }
+        }
+        s_lo *= kSwLog2e;
+        s_hi *= kSwLog2e;
         S[nt][j] = (in && sw_visible(qpos_lo, key, p.window, p.keep_first)) ? s_lo : -INFINITY;
         S[nt][2 + j] = (in && sw_visible(qpos_hi, key, p.window, p.keep_first)) ? s_hi : -INFINITY;
         mx_lo = fmaxf(mx_lo, S[nt][j]);
@@ -598,14 +643,17 @@ using namespace llmctl;
 
 // proj: [tokens, >= H*d + G*d + G*e] (row stride ld) = [q | k | v | ...]; bias: fp32 [H*d + G*d + G*e] or null; cache rows
 // have G*d + G*e numbers; slots = page * bs + offset, negative = not cached.
+// positions: null = no query temperature.
 LLMCTL_API int llmctl_window_kv_append(const void* proj, long long ld, const float* bias, int H, int G, int d, int e, int value_norm,
-                                       float eps, const long long* slots, float* q_out, void* cache, int tokens, int is_fp32,
-                                       void* stream) {
+                                       int qk_norm, float temp_coef, double temp_every, const int* positions, float eps,
+                                       const long long* slots, float* q_out, void* cache, int tokens, int is_fp32, void* stream) {
   LLMCTL_BEGIN();
+  LLMCTL_REQUIRE(positions == nullptr || temp_every > 0.0);
   LLMCTL_REQUIRE(H > 0 && G > 0 && d > 0 && e > 0 && ld >= static_cast<long long>(H + G) * d + static_cast<long long>(G) * e);
   if (tokens == 0) return 0;
   LLMCTL_DISPATCH_DTYPE(is_fp32, T, (window_kv_append_kernel<T><<<tokens, 256, 0, (cudaStream_t)stream>>>(
-                                        (const T*)proj, ld, bias, H, G, d, e, value_norm, eps, slots, q_out, (T*)cache)));
+                                        (const T*)proj, ld, bias, H, G, d, e, value_norm, qk_norm, temp_coef, temp_every, positions, eps, slots, q_out,
+                                        (T*)cache)));
   LLMCTL_RETURN_LAST();
 }
 
@@ -677,18 +725,20 @@ static int launch_softcap_attention(const SoftcapAttnParams& p, int ntiles, size
 // tile_tokens: most tokens in a tile (<= 16; the tensor-core kernel, use_mma, takes 1 or up to 128); splits > 1 needs
 // part_ml [ntiles * H/HB * splits * 64] and part_o [ntiles * H/HB * splits * 32 * e] (fp32) and, on the tensor-core
 // kernel, tile_tokens 1.  window 0: every earlier key is seen.  cap 0: no soft cap.
+// table: fp32 [H, table_len] or null.
 LLMCTL_API int llmctl_softcap_window_attention(const float* q, const void* cache, const int* block_tables, int max_blocks,
                                                const int* tiles, int ntiles, int tile_tokens, const int* positions, const void* gate,
-                                               long long gate_ld, const float* slopes, const float* sinks, float scale, float cap,
-                                               int window, int keep_first, int H, int G, int d, int e, int bs, void* out, int splits,
+                                               long long gate_ld, const float* slopes, const float* sinks, const float* table, int table_len,
+                                               float scale, float cap, int window, int keep_first, int H, int G, int d, int e, int bs, void* out, int splits,
                                                float* part_ml, float* part_o, int is_fp32, int use_mma, void* stream) {
   LLMCTL_BEGIN();
   LLMCTL_REQUIRE(H > 0 && G > 0 && H % G == 0 && d > 0 && e > 0 && e <= 512 && bs > 0 && tile_tokens >= 1 && window >= 0 &&
                  keep_first >= 0 && cap >= 0.f);
+  LLMCTL_REQUIRE(table == nullptr || table_len >= 1);
   LLMCTL_REQUIRE(splits >= 1 && (splits == 1 || (part_ml != nullptr && part_o != nullptr)));
   if (ntiles == 0) return 0;
   cudaStream_t s = (cudaStream_t)stream;
-  SoftcapAttnParams p{q, cache, block_tables, max_blocks, tiles, positions, gate, gate_ld, slopes, sinks, scale, cap, window, keep_first,
+  SoftcapAttnParams p{q, cache, block_tables, max_blocks, tiles, positions, gate, gate_ld, slopes, sinks, table, table_len, scale, cap, window, keep_first,
                       H, G, d, e, bs, llmctl_softcap_attention_heads_per_cta(H, G, tile_tokens, use_mma), out, splits, part_ml, part_o};
   LLMCTL_REQUIRE(p.HB >= 1);
   const int head_blocks = H / p.HB;

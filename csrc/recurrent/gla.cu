@@ -13,7 +13,8 @@
 //       CTA stages a chunk's prepared numbers and values in shared memory while the previous chunk's steps run on
 //       what was staged before; a step reads its rows' numbers as broadcast float4s.  The warps' partial outputs of a chunk meet in shared memory: two barriers per chunk, none per token.
 //       A portion that starts at position 0 starts from zeros whatever its slot holds; otherwise from the slot.
-//   llmctl_gla_output : per (token, head), o / sqrt(mean(o^2) + eps) * w (w shared by the heads) times silu(gate).
+//   llmctl_gla_output : per (token, head), o / sqrt(mean(o^2) + eps) * w (w shared by the heads, or one row per head) times
+//       silu(gate) or sigmoid(gate).
 // Decay, state, outputs and the norm are fp32; q, k, v, z and the gate are read in the projections' type.
 // Reference: none (the reference has no model code).
 #include "../common/dtype.cuh"
@@ -175,8 +176,8 @@ gla_scan_kernel(const GlaParams p, const float* __restrict__ work) {
 // one warp per (token, head)
 template <typename T>
 __global__ void __launch_bounds__(256)
-gla_output_kernel(const float* __restrict__ o, const float* __restrict__ w, const T* __restrict__ gate, long long ldg,
-                  T* __restrict__ out, long long rows, int H, int e, float eps) {
+gla_output_kernel(const float* __restrict__ o, const float* __restrict__ w, int w_stride, const T* __restrict__ gate, long long ldg,
+                  int gate_sigmoid, T* __restrict__ out, long long rows, int H, int e, float eps) {
   const long long r = blockIdx.x * static_cast<long long>(blockDim.x >> 5) + (threadIdx.x >> 5);
   if (r >= rows) return;
   const int lane = threadIdx.x & 31;
@@ -189,7 +190,7 @@ gla_output_kernel(const float* __restrict__ o, const float* __restrict__ w, cons
   const float f = 1.f / sqrtf(ss / e + eps);
   for (int c = lane; c < e; c += 32) {
     const float g = to_f32(gate[t * ldg + h * e + c]);
-    out[r * e + c] = from_f32<T>(orow[c] * f * w[c] * (g / (1.f + expf(-g))));
+    out[r * e + c] = from_f32<T>(orow[c] * f * w[h * w_stride + c] * ((gate_sigmoid ? 1.f : g) / (1.f + expf(-g))));
   }
 }
 
@@ -221,14 +222,15 @@ LLMCTL_API int llmctl_gla_scan(const void* q, long long ldq, const void* k, long
   LLMCTL_RETURN_LAST();
 }
 
-// o: fp32 [T, H * e]; w: fp32 [e]; gate: [T, H * e] (row stride ldg) pre-activation; out: [T, H * e] in the activation type.
-LLMCTL_API int llmctl_gla_output(const float* o, const float* w, const void* gate, long long ldg, void* out, int tokens, int H, int e,
-                                 float eps, int is_fp32, void* stream) {
+// o: fp32 [T, H * e]; w: fp32 [e] (w_stride 0) or [H, e] (w_stride e); gate: [T, H * e] (row stride ldg) pre-activation;
+// out: [T, H * e] in the activation type.
+LLMCTL_API int llmctl_gla_output(const float* o, const float* w, int w_stride, const void* gate, long long ldg, int gate_sigmoid, void* out,
+                                 int tokens, int H, int e, float eps, int is_fp32, void* stream) {
   LLMCTL_BEGIN();
   if (tokens == 0) return 0;
   const long long rows = static_cast<long long>(tokens) * H;
   const int grid = static_cast<int>((rows + 7) / 8);
-  LLMCTL_DISPATCH_DTYPE(is_fp32, T, (gla_output_kernel<T><<<grid, 256, 0, (cudaStream_t)stream>>>(o, w, (const T*)gate, ldg, (T*)out, rows,
+  LLMCTL_DISPATCH_DTYPE(is_fp32, T, (gla_output_kernel<T><<<grid, 256, 0, (cudaStream_t)stream>>>(o, w, w_stride, (const T*)gate, ldg, gate_sigmoid, (T*)out, rows,
                                                                                                 H, e, eps)));
   LLMCTL_RETURN_LAST();
 }

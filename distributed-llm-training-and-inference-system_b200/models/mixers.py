@@ -19,7 +19,8 @@ by element with the sigmoid of one more projection of the mixer's input (packed 
 ``SoftcapWindowAttention``: grouped-query attention without rotation whose scores pass a tanh soft cap and lose a linear
 distance bias with one slope per head; a sliding window that also keeps the first tokens of the sequence; a softmax with
 one added to the denominator (a sink of score 0); values cached at unit RMS per head; projection biases; a sigmoid output
-gate.  Every part is a field of ``SoftcapWindowAttentionSpec``.  Per step:
+gate; queries and keys at unit RMS per head; a query temperature that grows with the position; a learned bias per
+logarithmic distance bucket.  Every part is a field of ``SoftcapWindowAttentionSpec``.  Per step:
 
     p        = h Wp^T                           (one packed GEMM: q | k | v | gate)
     q, cache = bias / value norm / append       (ops.softcap_attention.window_kv_append)
@@ -61,6 +62,20 @@ decay GEMM, ``ops.recurrent.gla_scan``, ``ops.recurrent.gla_output``, the output
 ``dt = softplus(dt Wdt^T + b)``; ``S <- exp(dt A) S + dt u B``, ``y = (S C + D u) silu(z)``; output GEMM.  The state of a
 sequence is S and the last ``taps - 1`` inputs of the convolution.
 
+``DeltaRule``: gated delta rule with a matrix state per head.  q, k, v pass a short causal convolution and silu, q and k become
+unit vectors; ``S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q`` with one decay per head, or one per head and key row
+from a low-rank projection; heads are RMS-normed with one shared weight and gated (sigmoid of a low-rank projection, or silu
+of a full one).  Per step: one packed GEMM (q | k | v | latents or gate and decay | write strength), one block-diagonal GEMM for
+both low-rank projections, ``ops.matrix_state.delta_rule``, the output GEMM.
+
+``BonusMemory`` (RWKV-style time mixing): every projection reads its own mix of the token's and the previous token's input;
+``o = (S + diag(u) k v^T)^T r;  S <- diag(w) S + k v^T`` with a data-dependent decay per key row; heads RMS-normed, times a weight
+and a silu gate.  Per step: ``ops.matrix_state.token_shift``, one batched GEMM (r, k, v, gate), the low-rank decay (two GEMMs and
+a tanh), ``ops.matrix_state.bonus_memory``, the output GEMM.
+
+``BranchPair``: two mixers side by side on one input; its output is an ``ops.dual_norm.BranchSum`` that the residual update
+evaluates (each branch RMS-normed over the model width with a weight of its own, half their sum).
+
 Reference: none — the reference has no model code (reference llmctl/runtime/engine.py:119-140)."""
 from __future__ import annotations
 
@@ -74,10 +89,12 @@ import torch.nn as nn
 from ..ops import diff_attention as dops
 from ..ops import functional as ops
 from ..ops import latent_attention as lops
+from ..ops import matrix_state as mops
 from ..ops import recurrent as rops
 from ..ops import softcap_attention as sops
 from ..ops import window_attention as wops
-from ..ops.elementwise import rope_frequencies, sigmoid_gate_
+from ..ops.dual_norm import BranchSum
+from ..ops.elementwise import rope_frequencies, sigmoid_gate_, tanh_
 
 
 @dataclass
@@ -285,6 +302,10 @@ class SoftcapWindowAttentionSpec:
     value_norm: bool = True     # every value head is cached at unit RMS (no weight)
     bias: bool = True           # q, k, v and output projections have biases
     out_gate: bool = True       # heads * sigmoid(Wg h) before the output projection
+    qk_norm: bool = False       # queries and keys are brought to unit RMS per head (no weight)
+    q_temp: Optional[Tuple[float, float]] = None    # (coef, every): q *= 1 + coef ln(floor((p + 1) / every) + 1)
+    bias_rows: int = 0          # rows of a learned bias per distance bucket and head (0: none)
+    bias_max: float = 0.0       # distance at which the last bucket begins at the latest
 
     @property
     def cache_width(self) -> int:
@@ -310,9 +331,16 @@ class SoftcapWindowAttention(nn.Module):
         self.b_o = nn.Parameter(torch.zeros(width, **f32)) if s.bias else None
         self.register_buffer("slopes", sops.distance_slopes(s.heads).to(device) if s.distance_bias else None, persistent=False)
         self.register_buffer("sinks", torch.zeros(s.heads, **f32) if s.sink_one else None, persistent=False)
+        self.rel = nn.Parameter(torch.zeros(s.bias_rows, s.heads, **f32)) if s.bias_rows else None
+        self._table: Optional[torch.Tensor] = None          # the learned bias by distance, formed on first use
+
+    def bias_table(self) -> Optional[torch.Tensor]:
+        if self.rel is not None and (self._table is None or self._table.device != self.rel.device):
+            self._table = sops.bucket_bias_table(self.rel.detach(), self.spec.bias_max).to(self.rel.device)
+        return self._table
 
     def load(self, get, prefix: str) -> None:
-        """Checkpoint names under ``prefix``: q, k, v (+ ``.b`` biases), g, o (+ ``o.b``)."""
+        """Checkpoint names under ``prefix``: q, k, v (+ ``.b`` biases), g, rel ([rows, heads]), o (+ ``o.b``)."""
         s = self.spec
         with torch.no_grad():
             parts = [get(prefix + "q"), get(prefix + "k"), get(prefix + "v")] + ([get(prefix + "g")] if s.out_gate else [])
@@ -321,6 +349,9 @@ class SoftcapWindowAttention(nn.Module):
             if s.bias:
                 self.b_in.copy_(torch.cat([get(prefix + "q.b"), get(prefix + "k.b"), get(prefix + "v.b")], dim=0).float())
                 self.b_o.copy_(get(prefix + "o.b").float())
+            if self.rel is not None:
+                self.rel.copy_(get(prefix + "rel").float())
+        self._table = None
 
     def cache_shape(self, num_blocks: int, block_size: int) -> Tuple[int, ...]:
         return (num_blocks, block_size, self.spec.cache_width)
@@ -329,13 +360,15 @@ class SoftcapWindowAttention(nn.Module):
         """h: [T, W] in the activation type; ``cache``: this layer's [pages, bs, G (d + e)]."""
         s = self.spec
         p = ops.linear(h, self.w_in)
-        q = sops.window_kv_append(p, self.b_in, s.heads, s.kv_heads, s.dim, s.vdim, s.value_norm, self.eps, batch.slots, cache)
+        q = sops.window_kv_append(p, self.b_in, s.heads, s.kv_heads, s.dim, s.vdim, s.value_norm, self.eps, batch.slots, cache,
+                                  qk_norm=s.qk_norm, q_temp=s.q_temp, positions=batch.positions)
         gate = p[:, self.n_qkv:] if s.out_gate else None
         # prompt portions: tiles of 128 tokens on the tensor-core kernel, of 16 on the FMA kernel; decoded tokens: one each
         width = sops.tile_width(cache.dtype, s.heads, s.kv_heads, s.dim, s.vdim, q.is_cuda, batch.decode_only)
         o = sops.softcap_window_attention(q, cache, batch.block_tables, batch.tiles(width), 1 if batch.decode_only else width,
                                           batch.positions, gate, self.slopes, self.sinks, s.scale, s.softcap, s.window, s.keep_first,
-                                          s.heads, s.kv_heads, s.dim, s.vdim, batch.block_size, h.dtype, max_context=batch.max_context)
+                                          s.heads, s.kv_heads, s.dim, s.vdim, batch.block_size, h.dtype, max_context=batch.max_context,
+                                          table=self.bias_table())
         y = ops.linear(o, self.w_o)
         return y if self.b_o is None else torch.add(y, self.b_o)        # fp32 sum: the residual update takes either type
 
@@ -526,3 +559,181 @@ class SelectiveScan(nn.Module):
         dtp = ops.linear(bc[:, :R], self.w_dt)
         y = rops.selective_scan(u, bc, R, R + N, dtp, self.dt_bias, self.A, self.D, z, x, batch.portions, state[0], state[1])
         return ops.linear(y, self.w_o)
+
+
+def _pad8(n: int) -> int:
+    return (n + 7) // 8 * 8
+
+
+@dataclass
+class DeltaRuleSpec:
+    heads: int
+    kv_heads: int       # query / key heads: head h reads h // (heads // kv_heads)
+    dim: int            # query / key size per head
+    vdim: int           # value size per head
+    conv: int           # taps of the causal convolutions
+    per_channel: bool   # one decay per head and key row from a low-rank projection; otherwise one per head
+    decay_rank: int = 0     # inner size of the low-rank decay projection (per_channel)
+    gate_rank: int = 0      # inner size of a low-rank output gate; 0: full projection
+    gate_act: str = "silu"  # activation of the output gate: silu or sigmoid
+
+
+class DeltaRule(nn.Module):
+    stateful = True
+
+    def __init__(self, width: int, spec: DeltaRuleSpec, eps: float, dtype, device):
+        super().__init__()
+        s = self.spec = spec
+        if s.heads % s.kv_heads or s.conv < 1 or s.dim > mops.MAX_DIM or (s.per_channel and s.decay_rank < 1):
+            raise ValueError(f"inconsistent delta-rule sizes: {s}")
+        self.eps = eps
+        kw = dict(dtype=dtype, device=device)
+        f32 = dict(dtype=torch.float32, device=device)
+        H, nk, nv = s.heads, s.kv_heads * s.dim, s.heads * s.vdim
+        self.n_qkv = 2 * nk + nv
+        # rows of the packed projection: q, k, v without gaps (one convolution runs over them), then parts that start at
+        # multiples of 8 (a GEMM reads the latents in place)
+        parts = [("a1", s.decay_rank) if s.per_channel else ("a", H), ("g1", s.gate_rank) if s.gate_rank else ("g", nv), ("b", H)]
+        self.at: Dict[str, int] = {}
+        rows = _pad8(self.n_qkv)
+        for name, n in parts:
+            self.at[name] = rows
+            rows += _pad8(n)
+        self.w_in = nn.Parameter(torch.zeros(rows, width, **kw))
+        self.conv_w = nn.Parameter(torch.zeros(self.n_qkv, s.conv, **f32))
+        self.n_z = H * s.dim if s.per_channel else H
+        # low-rank second stages as one block-diagonal matrix over the neighbouring latents [a1 | g1]
+        self.low_rows = (self.n_z if s.per_channel else 0) + (nv if s.gate_rank else 0)
+        self.low_k = (_pad8(s.decay_rank) if s.per_channel else 0) + _pad8(s.gate_rank)
+        self.low_at = self.at["a1"] if s.per_channel else self.at.get("g1", 0)
+        self.w_low = nn.Parameter(torch.zeros(_pad8(self.low_rows), self.low_k, **kw)) if self.low_rows else None
+        self.dt_bias = nn.Parameter(torch.zeros(self.n_z, **f32))
+        self.speed = nn.Parameter(torch.ones(H, **f32))                                     # exp(A_log)
+        self.norm = nn.Parameter(torch.ones(s.vdim, **f32))
+        self.w_o = nn.Parameter(torch.empty(width, nv, **kw))
+
+    def load(self, get, prefix: str) -> None:
+        """Checkpoint names under ``prefix``: q, k, v (+ ``.conv``), b, A_log, dt_bias, a1 + a2 or a, g1 + g2 or g, norm, o."""
+        s = self.spec
+        with torch.no_grad():
+            self.w_in.zero_()
+            self.w_in[:self.n_qkv].copy_(torch.cat([get(prefix + n) for n in ("q", "k", "v")], dim=0))
+            for name, at in self.at.items():
+                w = get(prefix + name)
+                self.w_in[at:at + w.shape[0]].copy_(w)
+            self.conv_w.copy_(torch.cat([get(prefix + n + ".conv").float() for n in ("q", "k", "v")], dim=0))
+            if self.w_low is not None:
+                self.w_low.zero_()
+                r = k = 0
+                if s.per_channel:
+                    self.w_low[:self.n_z, :s.decay_rank].copy_(get(prefix + "a2"))
+                    r, k = self.n_z, _pad8(s.decay_rank)
+                if s.gate_rank:
+                    self.w_low[r:r + s.heads * s.vdim, k:k + s.gate_rank].copy_(get(prefix + "g2"))
+            self.dt_bias.copy_(get(prefix + "dt_bias").float())
+            self.speed.copy_(torch.exp(get(prefix + "A_log").float()))
+            self.norm.copy_(get(prefix + "norm").float())
+            self.w_o.copy_(get(prefix + "o"))
+
+    def state_shapes(self) -> Tuple[Tuple[int, ...], ...]:
+        s = self.spec
+        return ((s.heads, s.dim, s.vdim), (s.conv - 1, self.n_qkv))
+
+    def forward(self, h: torch.Tensor, batch, state) -> torch.Tensor:
+        """h: [T, W] in the activation type; ``state``: this layer run's ([slots, H, d, e], [slots, taps - 1, C]) fp32."""
+        s = self.spec
+        p = ops.linear(h, self.w_in)
+        low = ops.linear(p[:, self.low_at:self.low_at + self.low_k], self.w_low) if self.w_low is not None else None
+        nv = s.heads * s.vdim
+        z = low[:, :self.n_z] if s.per_channel else p[:, self.at["a"]:self.at["a"] + s.heads]
+        if s.gate_rank:
+            at = self.n_z if s.per_channel else 0
+            gate = low[:, at:at + nv]
+        else:
+            gate = p[:, self.at["g"]:self.at["g"] + nv]
+        y = mops.delta_rule(p[:, :self.n_qkv], self.conv_w, z, self.dt_bias, self.speed, p[:, self.at["b"]:self.at["b"] + s.heads], gate,
+                            self.norm, batch.portions, batch.seq_rows, state[0], state[1], s.heads, s.kv_heads, s.dim, s.vdim,
+                            s.per_channel, self.eps, s.gate_act, decode=batch.decode_only)
+        return ops.linear(y, self.w_o)
+
+
+@dataclass
+class BonusMemorySpec:
+    heads: int
+    dim: int            # key and value size per head
+    decay_rank: int     # inner size of the low-rank decay projection
+
+
+class BonusMemory(nn.Module):
+    stateful = True
+    MIXES = ("r", "k", "v", "g", "w")
+
+    def __init__(self, width: int, spec: BonusMemorySpec, eps: float, dtype, device):
+        super().__init__()
+        s = self.spec = spec
+        if s.dim > mops.MAX_DIM or s.decay_rank < 1:
+            raise ValueError(f"inconsistent time-mixing sizes: {s}")
+        self.eps = eps
+        kw = dict(dtype=dtype, device=device)
+        f32 = dict(dtype=torch.float32, device=device)
+        n = s.heads * s.dim
+        self.mu = nn.Parameter(torch.zeros(len(self.MIXES), width, **f32))
+        self.w_rkvg = nn.Parameter(torch.empty(4, n, width, **kw))
+        self.w_1 = nn.Parameter(torch.zeros(_pad8(s.decay_rank), width, **kw))
+        self.w_2 = nn.Parameter(torch.zeros(n, _pad8(s.decay_rank), **kw))
+        self.w_0 = nn.Parameter(torch.zeros(n, **f32))
+        self.u = nn.Parameter(torch.zeros(n, **f32))
+        self.norm = nn.Parameter(torch.ones(n, **f32))
+        self.w_o = nn.Parameter(torch.empty(width, n, **kw))
+
+    def load(self, get, prefix: str) -> None:
+        """Checkpoint names under ``prefix``: mu.{r,k,v,g,w}, r, k, v, g, w1, w2, w0, u ([heads, dim]), norm, o."""
+        r = self.spec.decay_rank
+        with torch.no_grad():
+            for i, name in enumerate(self.MIXES):
+                self.mu[i].copy_(get(prefix + "mu." + name).float())
+            for i, name in enumerate(self.MIXES[:4]):
+                self.w_rkvg[i].copy_(get(prefix + name))
+            self.w_1.zero_()
+            self.w_2.zero_()
+            self.w_1[:r].copy_(get(prefix + "w1"))
+            self.w_2[:, :r].copy_(get(prefix + "w2"))
+            self.w_0.copy_(get(prefix + "w0").float())
+            self.u.copy_(get(prefix + "u").float().reshape(-1))
+            self.norm.copy_(get(prefix + "norm").float())
+            self.w_o.copy_(get(prefix + "o"))
+
+    def state_shapes(self) -> Tuple[Tuple[int, ...], ...]:
+        s = self.spec
+        return ((s.heads, s.dim, s.dim), (self.mu.shape[1],))
+
+    def forward(self, h: torch.Tensor, batch, state) -> torch.Tensor:
+        """h: [T, W] in the activation type; ``state``: this layer run's ([slots, H, d, d], [slots, W]) fp32."""
+        s = self.spec
+        mix = mops.token_shift(h, self.mu, batch.portions, batch.seq_rows, state[1])
+        r, k, v, g = torch.bmm(mix[:4], self.w_rkvg.transpose(1, 2)).unbind(0)
+        z = ops.linear(tanh_(ops.linear(mix[4], self.w_1)), self.w_2)
+        y = mops.bonus_memory(r, k, v, z, self.w_0, self.u, g, self.norm, h, batch.portions, state[0], state[1], s.heads, s.dim, self.eps,
+                              decode=batch.decode_only)
+        return ops.linear(y, self.w_o)
+
+
+class BranchPair(nn.Module):
+    def __init__(self, width: int, left: nn.Module, right: nn.Module, device):
+        super().__init__()
+        self.left, self.right = left, right
+        f32 = dict(dtype=torch.float32, device=device)
+        self.left_w = nn.Parameter(torch.ones(width, **f32))
+        self.right_w = nn.Parameter(torch.ones(width, **f32))
+
+    def load(self, get, prefix: str) -> None:
+        """Checkpoint names under ``prefix``: left.*, right.* (the branches'), left.out, right.out."""
+        self.left.load(get, prefix + "left.")
+        self.right.load(get, prefix + "right.")
+        with torch.no_grad():
+            self.left_w.copy_(get(prefix + "left.out").float())
+            self.right_w.copy_(get(prefix + "right.out").float())
+
+    def forward(self, h: torch.Tensor, batch, own) -> BranchSum:
+        """``own``: (the left branch's cache or states, the right branch's)."""
+        return BranchSum(self.left(h, batch, own[0]), self.right(h, batch, own[1]), self.left_w, self.right_w, 0.5)

@@ -29,6 +29,7 @@ native.register_signature("llmctl_xielu", [c_void_p, c_void_p, c_int, c_ll, c_fl
 native.register_signature("llmctl_gated_silu", [c_void_p, c_ll, c_void_p, c_int, c_int, c_int, c_void_p])
 native.register_signature("llmctl_gated_gelu_tanh", [c_void_p, c_ll, c_void_p, c_int, c_int, c_int, c_void_p])
 native.register_signature("llmctl_sigmoid_gate", [c_void_p, c_void_p, c_ll, c_int, c_int, c_int, c_void_p])
+native.register_signature("llmctl_tanh", [c_void_p, c_ll, c_int, c_int, c_int, c_void_p])
 native.register_signature("llmctl_relu_squared", [c_void_p, c_void_p, c_int, c_ll, c_void_p])
 native.register_signature("llmctl_embed_positions", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p])
 native.register_signature("llmctl_rmsnorm_rows", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p])
@@ -184,6 +185,15 @@ def sigmoid_gate_(y: torch.Tensor, z: torch.Tensor) -> torch.Tensor:
         native.call("llmctl_sigmoid_gate", y.data_ptr(), z.data_ptr(), z.stride(0), _is32(y), rows, Fc, native.stream_ptr())
         return y
     return y.copy_((y.float() * torch.sigmoid(z.float())).to(y.dtype))
+
+
+def tanh_(z: torch.Tensor) -> torch.Tensor:
+    """``tanh(z)`` in place (fp32 inside); z: [rows, F], a view with unit column stride."""
+    assert z.dim() == 2 and z.stride(1) == 1
+    if z.is_cuda:
+        native.call("llmctl_tanh", z.data_ptr(), z.stride(0), _is32(z), z.shape[0], z.shape[1], native.stream_ptr())
+        return z
+    return z.copy_(torch.tanh(z.float()).to(z.dtype))
 
 
 def relu_squared(z: torch.Tensor) -> torch.Tensor:

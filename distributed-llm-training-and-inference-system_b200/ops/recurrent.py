@@ -25,7 +25,8 @@ c_void_p, c_int, c_ll, c_float = native.c_void_p, native.c_int, native.c_ll, nat
 native.register_signature("llmctl_gla_scan", [c_void_p, c_ll, c_void_p, c_ll, c_void_p, c_ll, c_void_p, c_ll, c_void_p, c_void_p, c_int, c_int,
                                                c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_float, c_int, c_void_p])
 native._KERNELS_PER_CALL["llmctl_gla_scan"] = 2
-native.register_signature("llmctl_gla_output", [c_void_p, c_void_p, c_void_p, c_ll, c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p])
+native.register_signature("llmctl_gla_output", [c_void_p, c_void_p, c_int, c_void_p, c_ll, c_int, c_void_p, c_int, c_int, c_int, c_float, c_int,
+                                                 c_void_p])
 native.register_signature("llmctl_causal_conv_silu", [c_void_p, c_ll, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                                                        c_int, c_int, c_int, c_void_p])
 native.register_signature("llmctl_selective_scan", [c_void_p, c_void_p, c_ll, c_int, c_int, c_void_p, c_ll, c_void_p, c_void_p, c_void_p,
@@ -61,19 +62,24 @@ def gla_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tensor,
     return out.reshape(T, H * e)
 
 
-def gla_output(o: torch.Tensor, w: torch.Tensor, gate: torch.Tensor, H: int, e: int, eps: float, out_dtype: torch.dtype) -> torch.Tensor:
-    """``o / sqrt(mean(o^2) + eps) * w * silu(gate)`` per (token, head); o: fp32 [T, H e]; w: fp32 [e]; gate: [T, H e]
-    pre-activation (unit column stride).  Returns [T, H e] in ``out_dtype``."""
+def gla_output(o: torch.Tensor, w: torch.Tensor, gate: torch.Tensor, H: int, e: int, eps: float, out_dtype: torch.dtype,
+               gate_act: str = "silu") -> torch.Tensor:
+    """``o / sqrt(mean(o^2) + eps) * w * act(gate)`` per (token, head); o: fp32 [T, H e]; w: fp32 [e] (shared by the heads) or
+    [H e]; gate: [T, H e] pre-activation (unit column stride); ``gate_act``: "silu" or "sigmoid".  Returns [T, H e] in
+    ``out_dtype``."""
     T = o.shape[0]
+    assert gate_act in ("silu", "sigmoid") and w.numel() in (e, H * e)
+    per_head = w.numel() != e
     if o.is_cuda:
         assert o.is_contiguous() and gate.stride(1) == 1 and gate.dtype == out_dtype
         out = torch.empty(T, H * e, dtype=out_dtype, device=o.device)
-        native.call("llmctl_gla_output", o.data_ptr(), w.data_ptr(), gate.data_ptr(), gate.stride(0), out.data_ptr(), T, H, e, float(eps),
-                    int(out_dtype == torch.float32), native.stream_ptr())
+        native.call("llmctl_gla_output", o.data_ptr(), w.data_ptr(), e if per_head else 0, gate.data_ptr(), gate.stride(0),
+                    int(gate_act == "sigmoid"), out.data_ptr(), T, H, e, float(eps), int(out_dtype == torch.float32), native.stream_ptr())
         return out
     oh = o.view(T, H, e)
-    y = oh / torch.sqrt(oh.pow(2).mean(-1, keepdim=True) + eps) * w
-    return (y.reshape(T, H * e) * F.silu(gate.float())).to(out_dtype)
+    y = oh / torch.sqrt(oh.pow(2).mean(-1, keepdim=True) + eps) * (w.view(H, e) if per_head else w)
+    g = gate.float()
+    return (y.reshape(T, H * e) * (F.silu(g) if gate_act == "silu" else torch.sigmoid(g))).to(out_dtype)
 
 
 def causal_conv_silu(x: torch.Tensor, w: torch.Tensor, wb: Optional[torch.Tensor], portions: torch.Tensor, seq_rows: torch.Tensor,

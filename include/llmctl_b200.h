@@ -329,8 +329,9 @@ int llmctl_gla_scan(const void* q, long long ldq, const void* k, long long ldk, 
                     long long ldz, const float* z_bias, const int* portions, int nportions, int tokens, float* state, float* out,
                     float* work /* fp32 [tokens, 3 H d] scratch */, int H, int d, int e, float q_scale, float tau, int is_fp32,
                     void* stream);
-int llmctl_gla_output(const float* o, const float* w, const void* gate, long long ldg, void* out, int tokens, int H, int e,
-                      float eps, int is_fp32, void* stream);
+/* w_stride 0: one weight row for all heads, e: one per head; gate_sigmoid 0: silu(gate), 1: sigmoid(gate). */
+int llmctl_gla_output(const float* o, const float* w, int w_stride, const void* gate, long long ldg, int gate_sigmoid, void* out,
+                      int tokens, int H, int e, float eps, int is_fp32, void* stream);
 int llmctl_causal_conv_silu(const void* x, long long ldx, const float* w, const float* wb, const int* portions,
                             const int* seq_rows, const float* conv_state, void* out, int tokens, int C, int taps, int is_fp32,
                             void* stream);
@@ -356,18 +357,48 @@ int llmctl_residual_norm_canon_small(const void* a, int a_is_fp32, long long lda
                                      int out_is_fp32, void* stream);
 int llmctl_gated_gelu_tanh(const void* gate_up, long long ld, void* out, int is_fp32, int rows, int F, void* stream);
 int llmctl_sigmoid_gate(void* y, const void* z, long long ldz, int is_fp32, int rows, int F, void* stream);
-/* fp32 biases (or null), optional unit-RMS norm of every value head; q -> fp32, [k | v] -> cache row. */
+/* fp32 biases (or null), optional unit-RMS norm of every value head and of every query / key head, query temperature
+ * 1 + coef ln(floor((p + 1) / every) + 1) where positions are given; q -> fp32, [k | v] -> cache row. */
 int llmctl_window_kv_append(const void* proj, long long ld, const float* bias, int H, int G, int d, int e, int value_norm,
-                            float eps, const long long* slots, float* q_out, void* cache, int tokens, int is_fp32, void* stream);
+                            int qk_norm, float temp_coef, double temp_every, const int* positions, float eps,
+                            const long long* slots, float* q_out, void* cache, int tokens, int is_fp32, void* stream);
 int llmctl_softcap_attention_heads_per_cta(int H, int G, int tile_tokens, int use_mma);
 int llmctl_softcap_attention_mma_ok(int H, int G, int d, int e, int tile_tokens);
 /* Sliding window (0: none) with kept first tokens, tanh soft cap (0: none), per-head distance slopes and sinks (null:
- * none), sigmoid output gate (null: none). */
+ * none), table of biases by distance [H, table_len] (null: none), sigmoid output gate (null: none). */
 int llmctl_softcap_window_attention(const float* q, const void* cache, const int* block_tables, int max_blocks, const int* tiles,
                                     int ntiles, int tile_tokens, const int* positions, const void* gate, long long gate_ld,
-                                    const float* slopes, const float* sinks, float scale, float cap, int window, int keep_first,
-                                    int H, int G, int d, int e, int bs, void* out, int splits, float* part_ml, float* part_o,
-                                    int is_fp32, int use_mma, void* stream);
+                                    const float* slopes, const float* sinks, const float* table, int table_len, float scale,
+                                    float cap, int window, int keep_first, int H, int G, int d, int e, int bs, void* out,
+                                    int splits, float* part_ml, float* part_o, int is_fp32, int use_mma, void* stream);
+
+/* ---- two-norm parallel layers, matrix-state recurrences (csrc/norm/dual_norm.cu, csrc/recurrent/matrix_state.cu) ---- */
+/* x += m + f [+ add] with m = a, or half_sum * (wa a / rms(a) + wb b / rms(b)); out_s = w_s x / rms(x), S = 0 .. 2. */
+int llmctl_residual_dual_norm(const void* a, long long lda, const void* b, long long ldb, const float* wa, const float* wb,
+                              float half_sum, const void* f, long long ldf, const float* add, float* x, int S, const float* w0,
+                              void* out0, const float* w1, void* out1, int rows, int W, float eps, int is_fp32, void* stream);
+/* x[t] = scale * table[tokens[t]] + sin / cos of positions[t] * freq; copy: a second fp32 copy or null. */
+int llmctl_embed_sinusoid(const long long* tokens, const int* positions, const void* table, int is_fp32, float scale,
+                          const double* freq, float* x, float* copy, int rows, int W, void* stream);
+/* kind 0: gated delta rule, one decay per head; 1: one per head and key row; 2: outer products with a bonus. */
+long long llmctl_matrix_scan_work(int tokens, int H, int G, int d, int e, int kind);
+int llmctl_delta_prepare(const void* x, long long ldx, const float* conv_w, const float* conv_state, int taps, const void* z,
+                         long long ldz, const float* dt_bias, const float* speed, const void* b, long long ldb, const int* portions,
+                         const int* seq_rows, int tokens, float* work, int H, int G, int d, int e, int kind, int is_fp32, void* stream);
+int llmctl_bonus_prepare(const void* r, long long ldr, const void* k, long long ldk, const void* v, long long ldv, const void* z,
+                         long long ldz, const float* w0, const float* u, int tokens, float* work, int H, int d, int is_fp32,
+                         void* stream);
+int llmctl_matrix_scan(float* work, const int* portions, int nportions, int tokens, float* state, float* out, int H, int G, int d, int e,
+                       int kind, const void* tail_x, long long tail_ld, int tail_C, int tail_keep, float* tail_state, int is_fp32,
+                       void* stream);
+int llmctl_matrix_step(const void* x, long long ldx, const void* r, long long ldr, const void* k, long long ldk, const void* v,
+                       long long ldv, const float* conv_w, float* conv_state, int taps, const void* z, long long ldz,
+                       const float* z_bias, const float* speed, const float* bonus, const void* b, long long ldb, const int* portions,
+                       int nportions, float* state, const float* norm_w, int norm_stride, const void* gate, long long ldg,
+                       int gate_kind, float eps, void* out, int H, int G, int d, int e, int kind, int is_fp32, void* stream);
+int llmctl_token_shift(const void* h, const float* mu, int n_mix, const int* portions, const int* seq_rows, float* state, void* out,
+                       int tokens, int W, int is_fp32, void* stream);
+int llmctl_tanh(void* z, long long ld, int is_fp32, int rows, int F, void* stream);
 
 #ifdef __cplusplus
 }
