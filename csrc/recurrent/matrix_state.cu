@@ -13,8 +13,8 @@
 //
 //   llmctl_delta_prepare / llmctl_bonus_prepare : fully parallel over tokens: convolutions, unit norms, step sizes, decays
 //       (minus one) and the per-token scalars, in fp32 and padded so that the scan copies whole 16-byte rows.
-//   llmctl_matrix_scan : the serial part.  A CTA owns (portion, head, 32 value columns).  LPC lanes share two columns, each
-//       with d / LPC rows of both in registers; a token costs one pass over them (decay, S^T k and S^T q together: the
+//   llmctl_matrix_scan : the serial part.  A CTA owns (portion, head, 16 or 32 value columns).  LPC lanes share one or two
+//       columns, each with d / LPC rows of them in registers; a token costs one pass over them (decay, S^T k and S^T q together: the
 //       read-out after the write is S_before^T q + (q . k) u), log2(LPC) shuffles and one update.  Products run as packed
 //       pairs (fma.rn.f32x2).  Chunks of 16 tokens are double-buffered in shared memory by cp.async.  At the end the CTAs of a
 //       portion also store its last raw inputs (the convolution's, or the previous token's row for kind 2's token shift).
@@ -34,8 +34,9 @@ __device__ __forceinline__ float ms_sigmoid(float x) { return 1.f / (1.f + expf(
 __device__ __forceinline__ float ms_silu(float x) { return x / (1.f + expf(-x)); }
 
 constexpr int kMsTC = 16;           // tokens per staged chunk of the scan
-constexpr int kMsCols = 32;         // value columns per CTA of the scan
-constexpr int kMsWalk = 16;         // consecutive tokens a warp of the prepare kernels walks
+constexpr int kMsCols = 32;         // most value columns per CTA of the scan
+constexpr int kMsNarrow = 148;      // up to this many CTAs of the wide scan: the narrow one runs
+constexpr int kMsWalk = 64;         // most consecutive tokens a warp of the delta prepare kernel walks
 
 static inline __host__ __device__ int ms_pad_rows(int d) { return d <= 32 ? 32 : d <= 64 ? 64 : d <= 128 ? 128 : 256; }
 static inline __host__ __device__ int ms_pad_cols(int e) { return (e + kMsCols - 1) / kMsCols * kMsCols; }
@@ -65,6 +66,7 @@ struct DeltaPrepParams {
   const int* portions;
   const int* seq_rows;
   int T, H, G, d, e, taps, kind;
+  int walk;                   // tokens per walk
   MsWork w;
 };
 
@@ -75,46 +77,60 @@ __device__ __forceinline__ float ms_raw(const T* x, long long ldx, long long src
   return st ? st[static_cast<long long>(keep - (t0 - src)) * C + c] : 0.f;
 }
 
-// Short convolution of one channel along consecutive tokens: up to four taps keep weights and history in registers,
-// longer ones read every tap again.
+// silu of a short convolution: bf16 inputs carry 8 bits, so the hardware's exponential and reciprocal are exact enough there
 template <typename T>
+__device__ __forceinline__ float ms_conv_act(float x) {
+  if (sizeof(T) == 2) return __fdividef(x, 1.f + __expf(-fmaxf(x, -80.f)));
+  return ms_silu(x);
+}
+
+// Short convolution of one channel along consecutive tokens.  SHORT (up to four taps): weights and history in registers;
+// otherwise every tap is read again.
+template <typename T, bool SHORT>
 struct ConvWalk {
-  float w[4], h[3];
+  float w[SHORT ? 4 : 1], h[SHORT ? 3 : 1];
   __device__ __forceinline__ void weights(const float* conv_w, int taps, int c) {
+    if (!SHORT) return;
+    if (taps == 4) {
+      const float4 v = *reinterpret_cast<const float4*>(conv_w + static_cast<long long>(c) * 4);
+      w[0] = v.x, w[SHORT ? 1 : 0] = v.y, w[SHORT ? 2 : 0] = v.z, w[SHORT ? 3 : 0] = v.w;
+      return;
+    }
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
+    for (int j = 0; j < (SHORT ? 4 : 0); ++j) {
       const int src = taps - 4 + j;                   // w[3] is the current token's weight
-      w[j] = (taps <= 4 && src >= 0) ? conv_w[static_cast<long long>(c) * taps + src] : 0.f;
+      w[j] = src >= 0 ? conv_w[static_cast<long long>(c) * taps + src] : 0.f;
     }
   }
   __device__ __forceinline__ void history(const T* x, long long ldx, long long t, int t0, const float* st, int taps, int C, int c) {
 #pragma unroll
-    for (int j = 0; j < 3; ++j) {
+    for (int j = 0; j < (SHORT ? 3 : 0); ++j) {
       const int back = 3 - j;
       h[j] = back <= taps - 1 ? ms_raw(x, ldx, t - back, t0, st, taps - 1, C, c) : 0.f;
     }
   }
-  __device__ __forceinline__ float step(const T* x, long long ldx, long long t, int t0, const float* st, const float* conv_w, int taps,
-                                        int C, int c) {
-    const float cur = to_f32(x[t * ldx + c]);
+  // cur: the channel's raw input of token t
+  __device__ __forceinline__ float step(float cur, const T* x, long long ldx, long long t, int t0, const float* st, const float* conv_w,
+                                        int taps, int C, int c) {
     float a;
-    if (taps <= 4) {
-      a = w[0] * h[0] + w[1] * h[1] + w[2] * h[2] + w[3] * cur;
-      h[0] = h[1];
-      h[1] = h[2];
-      h[2] = cur;
+    if (SHORT) {
+      a = w[0] * h[0] + w[SHORT ? 1 : 0] * h[SHORT ? 1 : 0] + w[SHORT ? 2 : 0] * h[SHORT ? 2 : 0] + w[SHORT ? 3 : 0] * cur;
+      h[0] = h[SHORT ? 1 : 0];
+      h[SHORT ? 1 : 0] = h[SHORT ? 2 : 0];
+      h[SHORT ? 2 : 0] = cur;
     } else {
       a = conv_w[static_cast<long long>(c) * taps + taps - 1] * cur;
       for (int j = 0; j < taps - 1; ++j)
         a += conv_w[static_cast<long long>(c) * taps + j] * ms_raw(x, ldx, t - (taps - 1 - j), t0, st, taps - 1, C, c);
     }
-    return ms_silu(a);
+    return ms_conv_act<T>(a);
   }
 };
 
 // A warp is one unit: units 0 .. G-1 are the query and key of a key/value head, then blocks of 128 padded value columns,
-// then (kind 1) blocks of 128 padded decay columns.  blockIdx.x: a walk of kMsWalk tokens.
-template <typename T, int NI>
+// then (kind 1) blocks of 128 padded decay columns.  blockIdx.x: a walk of p.walk tokens; the next token's raw inputs are
+// asked for before the current one's are used.
+template <typename T, int NI, bool SHORT>
 __global__ void __launch_bounds__(256)
 delta_prepare_kernel(const DeltaPrepParams p) {
   const int lane = threadIdx.x & 31;
@@ -123,45 +139,66 @@ delta_prepare_kernel(const DeltaPrepParams p) {
   const int nv = (H * ep + 127) / 128, nd = p.kind == 1 ? (H * dp + 127) / 128 : 0;
   int unit = blockIdx.y * 8 + (threadIdx.x >> 5);
   if (unit >= G + nv + nd) return;
-  const int tb = blockIdx.x * kMsWalk, te = min(tb + kMsWalk, p.T);
-  const T* x = static_cast<const T*>(p.x);
-  int prow = -1, t0 = 0;
+  const int tb = blockIdx.x * p.walk, te = min(tb + p.walk, p.T);
+  const T none = from_f32<T>(0.f);
+  int t0 = 0, t_end = -1;
   const float* st = nullptr;
   auto enter = [&](int t) {               // true when token t opens a portion (or the walk): histories are stale
-    const int r = p.seq_rows[t];
-    if (r == prow) return false;
-    prow = r;
-    const int* pt = p.portions + 4 * r;
+    if (t < t_end) return false;
+    const int* pt = p.portions + 4 * p.seq_rows[t];
     t0 = pt[0];
+    t_end = t0 + pt[1];
     st = (pt[2] > 0 && pt[3] >= 0) ? p.conv_state + static_cast<long long>(pt[3]) * keep * C : nullptr;
     return true;
   };
   if (unit < G) {
     const int g = unit;
-    ConvWalk<T> cq[NI], ck[NI];
+    const T* x = static_cast<const T*>(p.x);
+    ConvWalk<T, SHORT> cq[NI], ck[NI];
+    T nq[NI], nk[NI];
+    const T* row = x + tb * p.ldx + g * d + lane;
 #pragma unroll
     for (int i = 0; i < NI; ++i) {
       const int c = lane + 32 * i;
+      nq[i] = nk[i] = none;
       if (c < d) {
         cq[i].weights(p.conv_w, taps, g * d + c);
         ck[i].weights(p.conv_w, taps, (G + g) * d + c);
+        nq[i] = row[32 * i];
+        nk[i] = row[32 * i + G * d];
       }
     }
     const float qs = rsqrtf(static_cast<float>(d));
+#pragma unroll 1
     for (int t = tb; t < te; ++t) {
-      const bool fresh = enter(t);
       float q[NI], k[NI], sq = 0.f, sk = 0.f, qk = 0.f;
 #pragma unroll
-      for (int i = 0; i < NI; ++i) {
-        const int c = lane + 32 * i;
-        q[i] = k[i] = 0.f;
-        if (c < d) {
-          if (fresh && taps <= 4) {
+      for (int i = 0; i < NI; ++i) q[i] = to_f32(nq[i]), k[i] = to_f32(nk[i]);
+      row += p.ldx;
+      if (t + 1 < te) {
+#pragma unroll
+        for (int i = 0; i < NI; ++i)
+          if (lane + 32 * i < d) {
+            nq[i] = row[32 * i];
+            nk[i] = row[32 * i + G * d];
+          }
+      }
+      if (enter(t) && SHORT) {
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+          const int c = lane + 32 * i;
+          if (c < d) {
             cq[i].history(x, p.ldx, t, t0, st, taps, C, g * d + c);
             ck[i].history(x, p.ldx, t, t0, st, taps, C, (G + g) * d + c);
           }
-          q[i] = cq[i].step(x, p.ldx, t, t0, st, p.conv_w, taps, C, g * d + c);
-          k[i] = ck[i].step(x, p.ldx, t, t0, st, p.conv_w, taps, C, (G + g) * d + c);
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < NI; ++i) {
+        const int c = lane + 32 * i;
+        if (c < d) {
+          q[i] = cq[i].step(q[i], x, p.ldx, t, t0, st, p.conv_w, taps, C, g * d + c);
+          k[i] = ck[i].step(k[i], x, p.ldx, t, t0, st, p.conv_w, taps, C, (G + g) * d + c);
         }
         sq += q[i] * q[i];
         sk += k[i] * k[i];
@@ -169,12 +206,12 @@ delta_prepare_kernel(const DeltaPrepParams p) {
       }
       const float fq = qs / sqrtf(warp_sum(sq) + 1e-6f), fk = 1.f / sqrtf(warp_sum(sk) + 1e-6f);
       qk = warp_sum(qk) * fq * fk;
-      float* wq = p.w.q + (static_cast<long long>(t) * G + g) * dp;
-      float* wk = p.w.k + (static_cast<long long>(t) * G + g) * dp;
+      float* wq = p.w.q + (static_cast<long long>(t) * G + g) * dp + lane;
+      float* wk = p.w.k + (static_cast<long long>(t) * G + g) * dp + lane;
 #pragma unroll
       for (int i = 0; i < NI; ++i) {
-        wq[lane + 32 * i] = q[i] * fq;
-        wk[lane + 32 * i] = k[i] * fk;
+        wq[32 * i] = q[i] * fq;
+        wk[32 * i] = k[i] * fk;
       }
       for (int r = lane; r < rep; r += 32) {
         const int h = g * rep + r;
@@ -187,49 +224,60 @@ delta_prepare_kernel(const DeltaPrepParams p) {
     return;
   }
   unit -= G;
-  if (unit < nv) {
-    ConvWalk<T> cv[4];
-    int ch[4];
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const int col = unit * 128 + lane + 32 * i, h = col / ep, c = col % ep;
-      ch[i] = (h < H && c < e) ? 2 * G * d + h * e + c : -1;
-      if (ch[i] >= 0) cv[i].weights(p.conv_w, taps, ch[i]);
-    }
-    for (int t = tb; t < te; ++t) {
-      const bool fresh = enter(t);
-      float* wv = p.w.v + static_cast<long long>(t) * H * ep + unit * 128 + lane;
-#pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        float v = 0.f;
-        if (ch[i] >= 0) {
-          if (fresh && taps <= 4) cv[i].history(x, p.ldx, t, t0, st, taps, C, ch[i]);
-          v = cv[i].step(x, p.ldx, t, t0, st, p.conv_w, taps, C, ch[i]);
-        }
-        if (unit * 128 + lane + 32 * i < H * ep) wv[32 * i] = v;
-      }
-    }
-    return;
-  }
-  unit -= nv;
-  int zc[4];
+  const bool value = unit < nv;
+  if (!value) unit -= nv;
+  const int width = value ? ep : dp, real = value ? e : d;
+  const T* x = static_cast<const T*>(value ? p.x : p.z);
+  const long long ldx = value ? p.ldx : p.ldz;
+  float* out = (value ? p.w.v : p.w.dm) + static_cast<long long>(tb) * H * width + unit * 128 + lane;
+  ConvWalk<T, SHORT> cv[4];
+  int ch[4];
   float sp[4], bias[4];
+  T nx[4];
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
-    const int col = unit * 128 + lane + 32 * i, h = col / dp, c = col % dp;
-    const bool ok = h < H && c < d;
-    zc[i] = ok ? h * d + c : -1;
-    sp[i] = ok ? p.speed[h] : 0.f;
-    bias[i] = ok ? p.dt_bias[zc[i]] : 0.f;
-  }
-  for (int t = tb; t < te; ++t) {
-    float* wd = p.w.dm + static_cast<long long>(t) * H * dp + unit * 128 + lane;
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      float v = 0.f;
-      if (zc[i] >= 0) v = expm1f(-sp[i] * ms_softplus(to_f32(static_cast<const T*>(p.z)[static_cast<long long>(t) * p.ldz + zc[i]]) + bias[i]));
-      if (unit * 128 + lane + 32 * i < H * dp) wd[32 * i] = v;
+    const int col = unit * 128 + lane + 32 * i, h = col / width, c = col % width;
+    const bool ok = h < H && c < real;
+    ch[i] = ok ? (value ? 2 * G * d : 0) + h * real + c : -1;
+    sp[i] = bias[i] = 0.f;
+    nx[i] = none;
+    if (ok) {
+      nx[i] = x[tb * ldx + ch[i]];
+      if (value) {
+        cv[i].weights(p.conv_w, taps, ch[i]);
+      } else {
+        sp[i] = p.speed[h];
+        bias[i] = p.dt_bias[ch[i]];
+      }
     }
+  }
+#pragma unroll 1
+  for (int t = tb; t < te; ++t, out += H * width) {
+    float v[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) v[i] = to_f32(nx[i]);
+    if (t + 1 < te) {
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        if (ch[i] >= 0) nx[i] = x[(t + 1) * ldx + ch[i]];
+    }
+    if (value) {
+      if (enter(t) && SHORT) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+          if (ch[i] >= 0) cv[i].history(x, ldx, t, t0, st, taps, C, ch[i]);
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        if (ch[i] >= 0) v[i] = cv[i].step(v[i], x, ldx, t, t0, st, p.conv_w, taps, C, ch[i]);
+    } else {
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        if (ch[i] >= 0) v[i] = expm1f(-sp[i] * ms_softplus(v[i] + bias[i]));
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+      if (unit * 128 + lane + 32 * i < H * width) out[32 * i] = v[i];
   }
 }
 
@@ -320,27 +368,37 @@ struct MatrixScanParams {
   ScanTail tail;
 };
 
+// A token's prepared numbers as a lane holds them.
+template <int NP, int CPL, int KIND>
+struct ScanToken {
+  f32x2 k[NP], q[NP], d[KIND == 0 ? 1 : NP];
+  float4 sc;
+  float v[CPL];
+};
+
 // KIND 0: delta rule, decay per head; 1: delta rule, decay per key row; 2: outer products with a bonus.
-// A lane owns columns c0 and c0 + 1 and the rows (i LPC + sub) 4 .. + 3, i < RPT / 4.
-template <int RPT, int LPC, int KIND>
+// A lane owns columns c0 .. c0 + CPL - 1 and the rows (i LPC + sub) 4 .. + 3, i < RPT / 4; the CTA 16 CPL columns.
+template <int RPT, int LPC, int CPL, int KIND>
 __global__ void __launch_bounds__(LPC * 16)
 matrix_scan_kernel(const MatrixScanParams p) {
-  constexpr int TC = kMsTC, DP = RPT * LPC, NG = 32 / LPC, NT = LPC * 16, NP = RPT / 2;
-  constexpr int STAGE = TC * (DP * (KIND == 0 ? 2 : 3) + kMsCols + 4);
+  constexpr int TC = kMsTC, DP = RPT * LPC, NG = 32 / LPC, NT = LPC * 16, NP = RPT / 2, COLS = 16 * CPL;
+  constexpr int NROW = KIND == 0 ? 2 : 3, STAGE = TC * (DP * NROW + COLS + 4);
+  constexpr bool AHEAD = RPT <= 16;          // the next token's numbers are fetched while this one's sums meet
+  typedef ScanToken<NP, CPL, KIND> Tok;
   extern __shared__ __align__(16) float ms_smem[];
   const int H = p.H, d = p.d, e = p.e;
   const int* pt = p.portions + blockIdx.x * 4;
   const int t0 = pt[0], n = pt[1], pos0 = pt[2], slot = pt[3];
   if (n <= 0) return;
-  const int h = blockIdx.y, kvh = h / (H / p.G), ep = ms_pad_cols(e), cb = blockIdx.z * kMsCols;
+  const int h = blockIdx.y, kvh = h / (H / p.G), ep = ms_pad_cols(e), cb = blockIdx.z * COLS;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, sub = lane % LPC;
-  const int cl = (warp * NG + lane / LPC) * 2;               // first of this lane's columns within the CTA's
-  float* so = ms_smem + 2 * STAGE;                           // [2][TC][32] outputs of the chunk
+  const int cl = (warp * NG + lane / LPC) * CPL;             // first of this lane's columns within the CTA's
+  float* so = ms_smem + 2 * STAGE;                           // [2][TC][COLS] outputs of the chunk
 
-  f32x2 S[2][NP];
+  f32x2 S[CPL][NP];
   float* st = slot >= 0 ? p.state + ((static_cast<long long>(slot) * H + h) * d) * e : nullptr;
 #pragma unroll
-  for (int c = 0; c < 2; ++c)
+  for (int c = 0; c < CPL; ++c)
 #pragma unroll
     for (int j = 0; j < NP; ++j) {
       const int row = ((j >> 1) * LPC + sub) * 4 + (j & 1) * 2, col = cb + cl + c;
@@ -356,8 +414,8 @@ matrix_scan_kernel(const MatrixScanParams p) {
     float* sk = ms_smem + buf * STAGE;
     float* sq = sk + TC * DP;
     float* sd = sq + TC * DP;
-    float* sv = sk + TC * DP * (KIND == 0 ? 2 : 3);
-    float* ss = sv + TC * kMsCols;
+    float* sv = sk + TC * DP * NROW;
+    float* ss = sv + TC * COLS;
     const int cnt = min(TC, n - c0);
     const long long tb = t0 + c0;
     for (int i = tid; i < cnt * (DP / 4); i += NT) {
@@ -367,17 +425,18 @@ matrix_scan_kernel(const MatrixScanParams p) {
       cp_async_16(sq + tok * DP + c, p.w.q + src);
       if (KIND != 0) cp_async_16(sd + tok * DP + c, p.w.dm + ((tb + tok) * H + h) * DP + c);
     }
-    for (int i = tid; i < cnt * 9; i += NT) {
-      const int tok = i / 9, c = i % 9;
-      if (c < 8) cp_async_16(sv + tok * kMsCols + c * 4, p.w.v + ((tb + tok) * H + h) * ep + cb + c * 4);
+    constexpr int VC = COLS / 4;
+    for (int i = tid; i < cnt * (VC + 1); i += NT) {
+      const int tok = i / (VC + 1), c = i % (VC + 1);
+      if (c < VC) cp_async_16(sv + tok * COLS + c * 4, p.w.v + ((tb + tok) * H + h) * ep + cb + c * 4);
       else cp_async_16(ss + tok * 4, p.w.sc + ((tb + tok) * H + h) * 4);
     }
   };
-  auto flush = [&](int c0, int buf) {                        // the chunk's outputs, 32 neighbouring columns per token
+  auto flush = [&](int c0, int buf) {                        // the chunk's outputs, neighbouring columns of a token together
     const int cnt = min(TC, n - c0);
-    for (int i = tid; i < cnt * kMsCols; i += NT) {
-      const int tok = i / kMsCols, c = i % kMsCols;
-      if (cb + c < e) p.out[(static_cast<long long>(t0 + c0 + tok) * H + h) * e + cb + c] = so[(buf * TC + tok) * kMsCols + c];
+    for (int i = tid; i < cnt * COLS; i += NT) {
+      const int tok = i / COLS, c = i % COLS;
+      if (cb + c < e) p.out[(static_cast<long long>(t0 + c0 + tok) * H + h) * e + cb + c] = so[(buf * TC + tok) * COLS + c];
     }
   };
 
@@ -393,76 +452,94 @@ matrix_scan_kernel(const MatrixScanParams p) {
     const float* sk = ms_smem + buf * STAGE + sub * 4;
     const float* sq = sk + TC * DP;
     const float* sd = sq + TC * DP;
-    const float* sv = ms_smem + buf * STAGE + TC * DP * (KIND == 0 ? 2 : 3) + cl;
-    const float* ss = ms_smem + buf * STAGE + TC * DP * (KIND == 0 ? 2 : 3) + TC * kMsCols;
-    float* od = so + buf * TC * kMsCols + cl;
+    const float* sv = ms_smem + buf * STAGE + TC * DP * NROW + cl;
+    const float* ss = ms_smem + buf * STAGE + TC * DP * NROW + TC * COLS;
+    float* od = so + buf * TC * COLS + cl;
     const int cnt = min(TC, n - c0);
-#pragma unroll 1
-    for (int tok = 0; tok < cnt; ++tok) {
-      f32x2 k[NP], ka0 = 0ull, ka1 = 0ull, kb0 = 0ull, kb1 = 0ull, qa0 = 0ull, qa1 = 0ull, qb0 = 0ull, qb1 = 0ull;
-      const float4 sc = *reinterpret_cast<const float4*>(ss + tok * 4);
-      const float2 v = *reinterpret_cast<const float2*>(sv + tok * kMsCols);
-      const f32x2 dh = pk(sc.z, sc.z);
+
+    auto fetch = [&](Tok& w, int tok) {
+      w.sc = *reinterpret_cast<const float4*>(ss + tok * 4);
+#pragma unroll
+      for (int c = 0; c < CPL; ++c) w.v[c] = sv[tok * COLS + c];
 #pragma unroll
       for (int i = 0; i < NP; i += 2) {
-        f32x2 q0, q1, d0 = dh, d1 = dh;
-        ld_pairs(sk + tok * DP + i * 2 * LPC, k[i], k[i + 1]);
-        ld_pairs(sq + tok * DP + i * 2 * LPC, q0, q1);
-        if (KIND != 0) ld_pairs(sd + tok * DP + i * 2 * LPC, d0, d1);
-        if (KIND == 2) {                                     // the read-out sees the state before this token
-          qa0 = fma2(q0, S[0][i], qa0);
-          qa1 = fma2(q1, S[0][i + 1], qa1);
-          qb0 = fma2(q0, S[1][i], qb0);
-          qb1 = fma2(q1, S[1][i + 1], qb1);
+        ld_pairs(sk + tok * DP + i * 2 * LPC, w.k[i], w.k[i + 1]);
+        ld_pairs(sq + tok * DP + i * 2 * LPC, w.q[i], w.q[i + 1]);
+        if (KIND != 0) ld_pairs(sd + tok * DP + i * 2 * LPC, w.d[KIND == 0 ? 0 : i], w.d[KIND == 0 ? 0 : i + 1]);
+      }
+    };
+    auto step = [&](const Tok& w, Tok& next, int tok) {
+      f32x2 ka[CPL][2], qa[CPL][2];
+      const f32x2 dh = pk(w.sc.z, w.sc.z);
+#pragma unroll
+      for (int c = 0; c < CPL; ++c) ka[c][0] = ka[c][1] = qa[c][0] = qa[c][1] = 0ull;
+#pragma unroll
+      for (int i = 0; i < NP; ++i)
+#pragma unroll
+        for (int c = 0; c < CPL; ++c) {
+          if (KIND == 2) qa[c][i & 1] = fma2(w.q[i], S[c][i], qa[c][i & 1]);       // the read-out precedes this token's write
+          S[c][i] = fma2(KIND == 0 ? dh : w.d[KIND == 0 ? 0 : i], S[c][i], S[c][i]);
+          if (KIND != 2) ka[c][i & 1] = fma2(w.k[i], S[c][i], ka[c][i & 1]);
         }
-        S[0][i] = fma2(d0, S[0][i], S[0][i]);
-        S[0][i + 1] = fma2(d1, S[0][i + 1], S[0][i + 1]);
-        S[1][i] = fma2(d0, S[1][i], S[1][i]);
-        S[1][i + 1] = fma2(d1, S[1][i + 1], S[1][i + 1]);
+      float u[CPL], o[CPL];
+#pragma unroll
+      for (int c = 0; c < CPL; ++c) {
+        u[c] = w.v[c];
         if (KIND != 2) {
-          ka0 = fma2(k[i], S[0][i], ka0);
-          ka1 = fma2(k[i + 1], S[0][i + 1], ka1);
-          kb0 = fma2(k[i], S[1][i], kb0);
-          kb1 = fma2(k[i + 1], S[1][i + 1], kb1);
-          qa0 = fma2(q0, S[0][i], qa0);
-          qa1 = fma2(q1, S[0][i + 1], qa1);
-          qb0 = fma2(q0, S[1][i], qb0);
-          qb1 = fma2(q1, S[1][i + 1], qb1);
+          const float2 x = upk(ka[c][0]), y = upk(ka[c][1]);
+          o[c] = (x.x + y.x) + (x.y + y.y);
         }
       }
-      float ua = v.x, ub = v.y;
-      if (KIND != 2) {
-        const float2 a0 = upk(ka0), a1 = upk(ka1), b0 = upk(kb0), b1 = upk(kb1);
-        float ka = (a0.x + a1.x) + (a0.y + a1.y), kb = (b0.x + b1.x) + (b0.y + b1.y);
+      if (KIND != 2) {                       // the read-out's products fill the waits of these shuffles
 #pragma unroll
-        for (int o = LPC / 2; o > 0; o >>= 1) {
-          ka += __shfl_xor_sync(0xffffffffu, ka, o);
-          kb += __shfl_xor_sync(0xffffffffu, kb, o);
-        }
-        ua = sc.x * (v.x - ka);
-        ub = sc.x * (v.y - kb);
-      }
-      const f32x2 u0 = pk(ua, ua), u1 = pk(ub, ub);
+        for (int off = LPC / 2; off > 0; off >>= 1)
 #pragma unroll
-      for (int i = 0; i < NP; ++i) {
-        S[0][i] = fma2(k[i], u0, S[0][i]);
-        S[1][i] = fma2(k[i], u1, S[1][i]);
-      }
-      const float2 a0 = upk(qa0), a1 = upk(qa1), b0 = upk(qb0), b1 = upk(qb1);
-      float qa = (a0.x + a1.x) + (a0.y + a1.y), qb = (b0.x + b1.x) + (b0.y + b1.y);
+          for (int c = 0; c < CPL; ++c) o[c] += __shfl_xor_sync(0xffffffffu, o[c], off);
 #pragma unroll
-      for (int o = LPC / 2; o > 0; o >>= 1) {
-        qa += __shfl_xor_sync(0xffffffffu, qa, o);
-        qb += __shfl_xor_sync(0xffffffffu, qb, o);
+        for (int i = 0; i < NP; ++i)
+#pragma unroll
+          for (int c = 0; c < CPL; ++c) qa[c][i & 1] = fma2(w.q[i], S[c][i], qa[c][i & 1]);
+#pragma unroll
+        for (int c = 0; c < CPL; ++c) u[c] = w.sc.x * (w.v[c] - o[c]);
       }
-      if (sub == 0) *reinterpret_cast<float2*>(od + tok * kMsCols) = make_float2(qa + sc.y * ua, qb + sc.y * ub);
+      if (AHEAD) fetch(next, min(tok + 1, TC - 1));
+#pragma unroll
+      for (int c = 0; c < CPL; ++c) {
+        const f32x2 u2 = pk(u[c], u[c]);
+#pragma unroll
+        for (int i = 0; i < NP; ++i) S[c][i] = fma2(w.k[i], u2, S[c][i]);
+        const float2 x = upk(qa[c][0]), y = upk(qa[c][1]);
+        o[c] = (x.x + y.x) + (x.y + y.y);
+      }
+#pragma unroll
+      for (int off = LPC / 2; off > 0; off >>= 1)
+#pragma unroll
+        for (int c = 0; c < CPL; ++c) o[c] += __shfl_xor_sync(0xffffffffu, o[c], off);
+      if (sub == 0) {
+#pragma unroll
+        for (int c = 0; c < CPL; ++c) od[tok * COLS + c] = o[c] + w.sc.y * u[c];
+      }
+    };
+    Tok wa, wb;
+    if (AHEAD) {
+      fetch(wa, 0);
+      for (int tok = 0; tok < cnt; tok += 2) {
+        step(wa, wb, tok);
+        if (tok + 1 < cnt) step(wb, wa, tok + 1);
+      }
+    } else {
+#pragma unroll 1
+      for (int tok = 0; tok < cnt; ++tok) {
+        fetch(wa, tok);
+        step(wa, wa, tok);
+      }
     }
   }
   __syncthreads();
   flush((n - 1) / TC * TC, buf ^ 1);
   if (!st) return;
 #pragma unroll
-  for (int c = 0; c < 2; ++c)
+  for (int c = 0; c < CPL; ++c)
 #pragma unroll
     for (int j = 0; j < NP; ++j) {
       const int row = ((j >> 1) * LPC + sub) * 4 + (j & 1) * 2, col = cb + cl + c;
@@ -772,14 +849,29 @@ token_shift_vec_kernel(const T* __restrict__ h, const float* __restrict__ mu, in
   }
 }
 
+template <typename T, int NI>
+static void launch_delta_prepare(const DeltaPrepParams& p, dim3 grid, cudaStream_t s) {
+  if (p.taps <= 4) delta_prepare_kernel<T, NI, true><<<grid, 256, 0, s>>>(p);
+  else delta_prepare_kernel<T, NI, false><<<grid, 256, 0, s>>>(p);
+}
+
+template <int RPT, int LPC, int CPL, int KIND>
+static int launch_matrix_scan_cols(const MatrixScanParams& p, int nportions, cudaStream_t s) {
+  constexpr int DP = RPT * LPC, COLS = 16 * CPL;
+  const size_t smem = sizeof(float) * (2 * kMsTC * (static_cast<size_t>(DP) * (KIND == 0 ? 2 : 3) + COLS + 4) + 2 * kMsTC * COLS);
+  auto kern = matrix_scan_kernel<RPT, LPC, CPL, KIND>;
+  if (smem > 48 * 1024) LLMCTL_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
+  kern<<<dim3(nportions, p.H, (p.e + COLS - 1) / COLS), LPC * 16, smem, s>>>(p);
+  return 0;
+}
+
+// Two columns per lane share the loads of a token's vectors; with few CTAs a token's latency counts instead, and one
+// column per lane halves its work.
 template <int RPT, int LPC, int KIND>
 static int launch_matrix_scan(const MatrixScanParams& p, int nportions, cudaStream_t s) {
-  constexpr int DP = RPT * LPC;
-  const size_t smem = sizeof(float) * (2 * kMsTC * (static_cast<size_t>(DP) * (KIND == 0 ? 2 : 3) + kMsCols + 4) + 2 * kMsTC * kMsCols);
-  auto kern = matrix_scan_kernel<RPT, LPC, KIND>;
-  if (smem > 48 * 1024) LLMCTL_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
-  kern<<<dim3(nportions, p.H, ms_pad_cols(p.e) / kMsCols), LPC * 16, smem, s>>>(p);
-  return 0;
+  const long long ctas = static_cast<long long>(nportions) * p.H * (ms_pad_cols(p.e) / kMsCols);
+  return ctas <= kMsNarrow ? launch_matrix_scan_cols<RPT, LPC, 1, KIND>(p, nportions, s)
+                           : launch_matrix_scan_cols<RPT, LPC, 2, KIND>(p, nportions, s);
 }
 
 template <int KIND>
@@ -841,19 +933,22 @@ LLMCTL_API int llmctl_delta_prepare(const void* x, long long ldx, const float* c
                                     int kind, int is_fp32, void* stream) {
   LLMCTL_BEGIN();
   LLMCTL_REQUIRE(H > 0 && G > 0 && H % G == 0 && d > 0 && d <= 256 && e > 0 && taps >= 1 && (kind == 0 || kind == 1) && work != nullptr);
-  LLMCTL_REQUIRE((reinterpret_cast<uintptr_t>(work) & 15) == 0 && (taps == 1 || conv_state != nullptr));
+  LLMCTL_REQUIRE((reinterpret_cast<uintptr_t>(work) & 15) == 0 && (reinterpret_cast<uintptr_t>(conv_w) & 15) == 0);
+  LLMCTL_REQUIRE(taps == 1 || conv_state != nullptr);
   if (tokens == 0) return 0;
-  DeltaPrepParams p{x, ldx, conv_w, conv_state, z, ldz, dt_bias, speed, b, ldb, portions, seq_rows, tokens, H, G, d, e, taps, kind,
+  DeltaPrepParams p{x, ldx, conv_w, conv_state, z, ldz, dt_bias, speed, b, ldb, portions, seq_rows, tokens, H, G, d, e, taps, kind, kMsWalk,
                     ms_work(work, tokens, H, G, d, e, kind)};
   const int dp = ms_pad_rows(d), ep = ms_pad_cols(e);
   const int units = G + (H * ep + 127) / 128 + (kind == 1 ? (H * dp + 127) / 128 : 0);
-  const dim3 grid((tokens + kMsWalk - 1) / kMsWalk, (units + 7) / 8);
+  // long walks load weights and histories less often; short ones keep every SM busy
+  while (p.walk > 16 && ((tokens + p.walk - 1) / p.walk) * ((units + 7) / 8) < 2 * kNumSMs) p.walk /= 2;
+  const dim3 grid((tokens + p.walk - 1) / p.walk, (units + 7) / 8);
   cudaStream_t s = (cudaStream_t)stream;
   LLMCTL_DISPATCH_DTYPE(is_fp32, T, {
-    if (dp == 32) delta_prepare_kernel<T, 1><<<grid, 256, 0, s>>>(p);
-    else if (dp == 64) delta_prepare_kernel<T, 2><<<grid, 256, 0, s>>>(p);
-    else if (dp == 128) delta_prepare_kernel<T, 4><<<grid, 256, 0, s>>>(p);
-    else delta_prepare_kernel<T, 8><<<grid, 256, 0, s>>>(p);
+    if (dp == 32) launch_delta_prepare<T, 1>(p, grid, s);
+    else if (dp == 64) launch_delta_prepare<T, 2>(p, grid, s);
+    else if (dp == 128) launch_delta_prepare<T, 4>(p, grid, s);
+    else launch_delta_prepare<T, 8>(p, grid, s);
   });
   LLMCTL_RETURN_LAST();
 }

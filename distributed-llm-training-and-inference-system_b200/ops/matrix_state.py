@@ -57,6 +57,40 @@ def _gate_kind(act: str) -> int:
     return {"silu": 0, "sigmoid": 1}[act]
 
 
+def delta_prepare(qkv: torch.Tensor, conv_w: torch.Tensor, z: torch.Tensor, dt_bias: torch.Tensor, speed: torch.Tensor, b: torch.Tensor,
+                  portions: torch.Tensor, seq_rows: torch.Tensor, conv_state: torch.Tensor, H: int, G: int, d: int, e: int,
+                  kind: int) -> torch.Tensor:
+    """The parallel pass before a delta-rule scan (CUDA tensors, arguments as in ``delta_rule``); returns the scan's scratch."""
+    T, taps = qkv.shape[0], conv_w.shape[1]
+    work = torch.empty(work_numbers(T, H, G, d, e, kind), dtype=torch.float32, device=qkv.device)
+    native.call("llmctl_delta_prepare", qkv.data_ptr(), qkv.stride(0), conv_w.data_ptr(), conv_state.data_ptr() if taps > 1 else None, taps,
+                z.data_ptr(), z.stride(0), dt_bias.data_ptr(), speed.data_ptr(), b.data_ptr(), b.stride(0), portions.data_ptr(),
+                seq_rows.data_ptr(), T, work.data_ptr(), H, G, d, e, kind, _is32(qkv), native.stream_ptr())
+    return work
+
+
+def bonus_prepare(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tensor, w0: torch.Tensor, u: torch.Tensor, H: int,
+                  d: int) -> torch.Tensor:
+    """The parallel pass before a bonus-memory scan (CUDA tensors, arguments as in ``bonus_memory``); returns the scan's scratch."""
+    T = r.shape[0]
+    work = torch.empty(work_numbers(T, H, H, d, d, BONUS), dtype=torch.float32, device=r.device)
+    native.call("llmctl_bonus_prepare", r.data_ptr(), r.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), z.data_ptr(), z.stride(0),
+                w0.data_ptr(), u.data_ptr(), T, work.data_ptr(), H, d, _is32(r), native.stream_ptr())
+    return work
+
+
+def matrix_scan(work: torch.Tensor, portions: torch.Tensor, state: torch.Tensor, T: int, H: int, G: int, d: int, e: int, kind: int,
+                tail: torch.Tensor, tail_state: torch.Tensor) -> torch.Tensor:
+    """The serial pass over prepared tokens (CUDA tensors): updates ``state``, stores the last rows of ``tail`` [T, C] into
+    ``tail_state`` [slots, keep, C] and returns o, fp32 [T, H e]."""
+    o = torch.empty(T, H * e, dtype=torch.float32, device=work.device)
+    keep = tail_state.shape[1]
+    native.call("llmctl_matrix_scan", work.data_ptr(), portions.data_ptr(), portions.shape[0], T, state.data_ptr(), o.data_ptr(), H, G, d, e, kind,
+                tail.data_ptr(), tail.stride(0), tail.shape[1], keep, tail_state.data_ptr() if keep else None, _is32(tail),
+                native.stream_ptr())
+    return o
+
+
 def delta_rule(qkv: torch.Tensor, conv_w: torch.Tensor, z: torch.Tensor, dt_bias: torch.Tensor, speed: torch.Tensor, b: torch.Tensor,
                gate: torch.Tensor, norm_w: torch.Tensor, portions: torch.Tensor, seq_rows: torch.Tensor, state: torch.Tensor,
                conv_state: torch.Tensor, H: int, G: int, d: int, e: int, per_channel: bool, eps: float, gate_act: str,
@@ -81,13 +115,8 @@ def delta_rule(qkv: torch.Tensor, conv_w: torch.Tensor, z: torch.Tensor, dt_bias
                         portions.shape[0], state.data_ptr(), norm_w.data_ptr(), 0, gate.data_ptr(), gate.stride(0), _gate_kind(gate_act),
                         float(eps), out.data_ptr(), H, G, d, e, kind, _is32(qkv), native.stream_ptr())
             return out
-        work = torch.empty(work_numbers(T, H, G, d, e, kind), dtype=torch.float32, device=qkv.device)
-        native.call("llmctl_delta_prepare", qkv.data_ptr(), qkv.stride(0), conv_w.data_ptr(), cs, taps, z.data_ptr(), z.stride(0),
-                    dt_bias.data_ptr(), speed.data_ptr(), b.data_ptr(), b.stride(0), portions.data_ptr(), seq_rows.data_ptr(), T,
-                    work.data_ptr(), H, G, d, e, kind, _is32(qkv), native.stream_ptr())
-        o = torch.empty(T, H * e, dtype=torch.float32, device=qkv.device)
-        native.call("llmctl_matrix_scan", work.data_ptr(), portions.data_ptr(), portions.shape[0], T, state.data_ptr(), o.data_ptr(), H, G,
-                    d, e, kind, qkv.data_ptr(), qkv.stride(0), C, taps - 1, cs, _is32(qkv), native.stream_ptr())
+        work = delta_prepare(qkv, conv_w, z, dt_bias, speed, b, portions, seq_rows, conv_state, H, G, d, e, kind)
+        o = matrix_scan(work, portions, state, T, H, G, d, e, kind, qkv, conv_state)
         return gla_output(o, norm_w, gate, H, e, eps, qkv.dtype, gate_act)
     rep = H // G
     xf, keep = qkv.float(), taps - 1
@@ -137,12 +166,8 @@ def bonus_memory(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Ten
                         state.data_ptr(), norm_w.data_ptr(), d, gate.data_ptr(), gate.stride(0), _gate_kind(gate_act), float(eps),
                         out.data_ptr(), H, H, d, d, BONUS, _is32(r), native.stream_ptr())
             return out
-        work = torch.empty(work_numbers(T, H, H, d, d, BONUS), dtype=torch.float32, device=r.device)
-        native.call("llmctl_bonus_prepare", r.data_ptr(), r.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), z.data_ptr(),
-                    z.stride(0), w0.data_ptr(), u.data_ptr(), T, work.data_ptr(), H, d, _is32(r), native.stream_ptr())
-        o = torch.empty(T, H * d, dtype=torch.float32, device=r.device)
-        native.call("llmctl_matrix_scan", work.data_ptr(), portions.data_ptr(), portions.shape[0], T, state.data_ptr(), o.data_ptr(), H, H,
-                    d, d, BONUS, h.data_ptr(), h.stride(0), W, 1, shift_state.data_ptr(), _is32(r), native.stream_ptr())
+        work = bonus_prepare(r, k, v, z, w0, u, H, d)
+        o = matrix_scan(work, portions, state, T, H, H, d, d, BONUS, h, shift_state[:, None])
         return gla_output(o, norm_w, gate, H, d, eps, r.dtype, gate_act)
     w = torch.exp(-torch.exp(z.float() + w0)).view(T, H, d)
     rf, kf, vf, uf = r.float().reshape(T, H, d), k.float().reshape(T, H, d), v.float().reshape(T, H, d), u.view(H, d)

@@ -1,9 +1,9 @@
-"""Serving throughput of a ragged-batch design (Nafazen, Teluzen, Namisun, Tupidra) beside the GPT/LLaMA family at equal parameter count:
+"""Serving throughput of a ragged-batch design (Nafazen, Teluzen, Namisun, Tupidra, Zokepel) beside the GPT/LLaMA family at equal parameter count:
 prefill and decode tokens/s through ``InferenceEngine.generate`` (the scheduler, block manager and step function a
 user gets), random weights, a few layer sizes that resemble real models; plus device-timed runs of the design's own
 attention and expert kernels against the measured roofline, next to the GPT family's like kernels.
-``bench.py --arch-compare nafazen|teluzen|namisun|tupidra`` prints the result as one JSON line.  Tupidra is also set beside
-Namisun (the other parallel-layout design with state slots) of equal width and depth, with both designs' like kernels.
+``bench.py --arch-compare nafazen|teluzen|namisun|tupidra|zokepel`` prints the result as one JSON line.  Tupidra and Zokepel are
+also set beside Namisun (another parallel-layout design with state slots) of equal width and depth, with both designs' like kernels.
 
 Reference: the reference's serving benchmark is ``llmctl bench e2e`` (reference llmctl/cli/commands/bench.py:98-160)."""
 from __future__ import annotations
@@ -60,6 +60,22 @@ TUPIDRA_SIZES: Dict[str, Dict[str, Any]] = {
     "w4096": dict(width=4096, vocab=32000, pattern="MLAMcA", ff="1", taps=4, heads=32, kv_heads=8, dim=128, vdim=128, softcap=30.0,
                   window=512, keep_first=8, lat_heads=32, lat_dim=128, rot_dim=64, lat_vdim=128, kv_rank=512, q_rank=1536, inner=8192,
                   state=16, dt_rank=256, conv=4, ff_size=16384),
+}
+
+
+ZOKEPEL_SIZES: Dict[str, Dict[str, Any]] = {
+    # 6 layers: delta rule with a decay per key row, delta rule with a decay per head, attention beside time mixing, twice; a
+    # clamped gated feed-forward beside every mixer.  No loop here: a looped range adds compute without parameters, and the
+    # models beside it have equal parameters.
+    "w1024": dict(width=1024, vocab=32000, pattern="CDPCDP", ff="1", loop=None, heads=8, kv_heads=8, dim=128, vdim=128, conv=4, decay_rank=64,
+                  gate_rank=64, att_heads=8, att_kv_heads=2, att_dim=128, att_vdim=128, bias_rows=32, bias_max=256.0, q_temp=(0.1, 1024),
+                  mix_heads=16, mix_dim=64, mix_rank=64, ff_size=4096, limit=7.0),
+    "w2048": dict(width=2048, vocab=32000, pattern="CDPCDP", ff="1", loop=None, heads=16, kv_heads=16, dim=128, vdim=128, conv=4, decay_rank=128,
+                  gate_rank=128, att_heads=16, att_kv_heads=4, att_dim=128, att_vdim=128, bias_rows=32, bias_max=256.0, q_temp=(0.1, 1024),
+                  mix_heads=32, mix_dim=64, mix_rank=64, ff_size=8192, limit=7.0),
+    "w4096": dict(width=4096, vocab=32000, pattern="CDPCDP", ff="1", loop=None, heads=32, kv_heads=32, dim=128, vdim=128, conv=4, decay_rank=128,
+                  gate_rank=128, att_heads=32, att_kv_heads=8, att_dim=128, att_vdim=128, bias_rows=32, bias_max=256.0, q_temp=(0.1, 1024),
+                  mix_heads=64, mix_dim=64, mix_rank=128, ff_size=12288, limit=7.0),
 }
 
 
@@ -472,6 +488,138 @@ def _tupidra_kernels(size: Dict[str, Any], peaks: Dict[str, float]) -> Dict[str,
     return res
 
 
+def _zokepel_kernels(size: Dict[str, Any], peaks: Dict[str, float]) -> Dict[str, Any]:
+    """The design's own kernels in isolation (bf16, L2 flushed before every call; prefill 2 x 2048 tokens, decode 32 sequences,
+    context 4096 for the attention), each next to the like kernel of the closest design at the same sizes: attention with a
+    bias table against the same attention with Tupidra's cap, slopes, sink and gate and against Namisun's differential attention;
+    norms + temperature + append against Tupidra's bias + value norm + append; the matrix-state scans (with their prepare passes)
+    and single-launch decoding steps against Namisun's gated linear attention; the glue against Namisun's residual + layer norm;
+    the clamped gate against the gated SiLU."""
+    from ..ops import diff_attention as DA
+    from ..ops import dual_norm as D
+    from ..ops import elementwise as E
+    from ..ops import matrix_state as M
+    from ..ops import native
+    from ..ops import recurrent as R
+    from ..ops import softcap_attention as SA
+    from .ragged import Portion, RaggedBatch
+    dev = torch.device("cuda")
+    bf = torch.bfloat16
+    W, F = size["width"], size["ff_size"]
+    H, G, d, e, taps = size["heads"], size["kv_heads"], size["dim"], size["vdim"], size["conv"]
+    aH, aG, ad, ae = size["att_heads"], size["att_kv_heads"], size["att_dim"], size["att_vdim"]
+    mH, md = size["mix_heads"], size["mix_dim"]
+    bs, res = 64, {}
+    Wc = aG * (ad + ae)
+    table = SA.bucket_bias_table(torch.randn(size["bias_rows"], aH), size["bias_max"]).to(dev)
+    slopes, sinks = SA.distance_slopes(aH).to(dev), torch.zeros(aH, device=dev)
+
+    def hbm(key: str, t: float, bytes_: float, **more) -> None:
+        res[key] = {"ms": t * 1e3, "gbs": bytes_ / t / 1e9, "frac_of_hbm": bytes_ / t / 1e9 / peaks["hbm_gbs"], **more}
+
+    for name, nseq, ctx, new in (("prefill", 2, 2048, 2048), ("decode", 32, 4096, 1)):
+        per = (ctx + bs - 1) // bs
+        cache = torch.randn(nseq * per, bs, Wc, device=dev).to(bf)
+        ps = [Portion(i, [0] * new, ctx - new, [], list(range(i * per, (i + 1) * per)), i) for i in range(nseq)]
+        b = RaggedBatch(ps, bs, dev)
+        T = b.num_tokens
+        # attention
+        q = torch.randn(T, aH * ad, device=dev)
+        gate = torch.randn(T, aH * ae, device=dev).to(bf)
+        width = SA.tile_width(bf, aH, aG, ad, ae, True, new == 1)
+        tile = 1 if new == 1 else width
+        pairs = nseq * sum(i + 1 for i in range(ctx - new, ctx))
+        flops = 2.0 * aH * pairs * (ad + ae)
+        bytes_ = nseq * ctx * Wc * 2 + T * aH * (ad * 4 + ae * 2)
+        for key, kw, cap, gt, sl, sk in ((f"biased_attention_{name}", dict(table=table), 0.0, None, None, None),
+                                         (f"tupidra_softcap_attention_{name}", {}, 30.0, gate, slopes, sinks)):
+            t = _time_flushed(lambda: SA.softcap_window_attention(q, cache, b.block_tables, b.tiles(width), tile, b.positions, gt, sl, sk, ad ** -0.5,
+                                                                  cap, 0, 0, aH, aG, ad, ae, bs, bf, max_context=b.max_context, **kw))
+            hbm(key, t, bytes_, tflops=flops / t / 1e12, frac_of_bf16_peak=flops / t / 1e12 / peaks["bf16_tflops"])
+        nd = ad // 2
+        nq, ngate = torch.randn(T, aH * 2 * nd, device=dev), torch.randn(T, aH, device=dev).to(bf)
+        nwidth = DA.tile_width(bf, aH, aG, nd, ae, True, new == 1)
+        t = _time_flushed(lambda: DA.diff_attention(nq, cache, b.block_tables, b.tiles(nwidth), 1 if new == 1 else nwidth, b.positions, ngate, nd ** -0.5,
+                                                    0.5, 0.7, 1e-5, aH, aG, nd, ae, bs, bf, max_context=b.max_context))
+        nflops = 2.0 * aH * pairs * (2 * nd + 2 * ae)
+        hbm(f"namisun_diff_attention_{name}", t, bytes_, tflops=nflops / t / 1e12, frac_of_bf16_peak=nflops / t / 1e12 / peaks["bf16_tflops"])
+        # recurrences
+        C = 2 * G * d + H * e
+        decode = new == 1
+        p = torch.randn(T, C + H * d + H * e + H, device=dev).to(bf)
+        qkv, zc, gt, bb = p[:, :C], p[:, C:C + H * d], p[:, C + H * d:C + H * d + H * e], p[:, C + H * d + H * e:]
+        conv_w, speed, nw = torch.randn(C, taps, device=dev), torch.rand(H, device=dev), torch.ones(e, device=dev)
+        state, conv = torch.zeros(nseq, H, d, e, device=dev), torch.zeros(nseq, taps - 1, C, device=dev)
+        for key, ch in (("channel_delta", True), ("delta", False)):
+            z = zc if ch else bb
+            dtb = torch.rand(z.shape[1], device=dev) - 4.0
+            kind = M.DELTA_PER_CHANNEL if ch else M.DELTA_PER_HEAD
+            t_all = _time_flushed(lambda: M.delta_rule(qkv, conv_w, z, dtb, speed, bb, gt, nw, b.portions, b.seq_rows, state, conv, H, G, d, e, ch, 1e-6,
+                                                       "sigmoid", decode=decode))
+            bytes_ = T * 2 * (C + z.shape[1] + H + 2 * H * e) + 2 * 4 * (state.numel() + conv.numel())
+            more = {}
+            if not decode:
+                work = M.delta_prepare(qkv, conv_w, z, dtb, speed, bb, b.portions, b.seq_rows, conv, H, G, d, e, kind)
+                more["ms_prepare"] = 1e3 * _time_flushed(lambda: M.delta_prepare(qkv, conv_w, z, dtb, speed, bb, b.portions, b.seq_rows, conv, H, G, d, e,
+                                                                                kind))
+                more["ms_scan"] = 1e3 * _time_flushed(lambda: M.matrix_scan(work, b.portions, state, T, H, G, d, e, kind, qkv, conv))
+            hbm(f"{key}_{name}", t_all, bytes_, **more)
+        r5 = torch.randn(5, T, mH * md, device=dev).to(bf)
+        h = torch.randn(T, W, device=dev).to(bf)
+        mstate, shift = torch.zeros(nseq, mH, md, md, device=dev), torch.zeros(nseq, W, device=dev)
+        w0, u, mnw = torch.rand(mH * md, device=dev) - 4.0, torch.randn(mH * md, device=dev), torch.ones(mH * md, device=dev)
+        t = _time_flushed(lambda: M.bonus_memory(r5[0], r5[1], r5[2], r5[3], w0, u, r5[4], mnw, h, b.portions, mstate, shift, mH, md, 1e-6, decode=decode))
+        more = {}
+        if not decode:
+            work = M.bonus_prepare(r5[0], r5[1], r5[2], r5[3], w0, u, mH, md)
+            more["ms_prepare"] = 1e3 * _time_flushed(lambda: M.bonus_prepare(r5[0], r5[1], r5[2], r5[3], w0, u, mH, md))
+            more["ms_scan"] = 1e3 * _time_flushed(lambda: M.matrix_scan(work, b.portions, mstate, T, mH, mH, md, md, M.BONUS, h, shift[:, None]))
+        hbm(f"bonus_memory_{name}", t, T * 2 * 6 * mH * md + 2 * 4 * mstate.numel(), **more)
+        mu = torch.rand(5, W, device=dev)
+        t = _time_flushed(lambda: M.token_shift(h, mu, b.portions, b.seq_rows, shift))
+        hbm(f"token_shift_{name}", t, T * W * 2 * 6)
+        # Namisun's gated linear attention (scan with its prepare pass, head norm) at the sizes of either recurrence
+        for key, gH, gd, ge in (("128", H, d, e), ("64", mH, md, md)):
+            nk, nv = gH * gd, gH * ge
+            gp, gz = torch.randn(T, 2 * nk + 2 * nv, device=dev).to(bf), torch.randn(T, nk, device=dev).to(bf)
+            gzb, gst, gnw = torch.rand(nk, device=dev) * 4, torch.zeros(nseq, gH, gd, ge, device=dev), torch.ones(ge, device=dev)
+
+            def gla():
+                o = R.gla_scan(gp[:, :nk], gp[:, nk:2 * nk], gp[:, 2 * nk:2 * nk + nv], gz, gzb, b.portions, gst, gH, gd, ge, gd ** -0.5, 16.0)
+                return R.gla_output(o, gnw, gp[:, 2 * nk + nv:], gH, ge, 1e-6, bf)
+            hbm(f"namisun_gla_{key}_{name}", _time_flushed(gla), T * 2 * (3 * nk + 3 * nv) + 2 * 4 * gst.numel())
+        # glue
+        x, x0 = torch.randn(T, W, device=dev), torch.randn(T, W, device=dev)
+        a, a2, f = (torch.randn(T, W, device=dev).to(bf) for _ in range(3))
+        ws = [torch.ones(W, device=dev) for _ in range(4)]
+        t = _time_flushed(lambda: D.residual_dual_norm(a, f, x, 1e-6, ws[:2], bf))
+        hbm(f"residual_dual_norm_{name}", t, T * W * (2 + 2 + 4 + 4 + 2 + 2))
+        t = _time_flushed(lambda: D.residual_dual_norm(D.BranchSum(a, a2, ws[2], ws[3]), f, x, 1e-6, ws[:2], bf))
+        hbm(f"residual_dual_norm_branches_{name}", t, T * W * (2 + 2 + 2 + 4 + 4 + 2 + 2))
+        f32 = torch.randn(T, W, device=dev)
+        t = _time_flushed(lambda: E.parallel_residual(a, f32, x, 0.5, 1e-5, bf, ws[0], ws[1], want_fp32=True))
+        hbm(f"namisun_residual_norm_{name}", t, T * W * (2 + 4 + 4 + 4 + 2 + 4))
+        if new > 1:
+            tab = torch.randn(32000, W, device=dev).to(bf)
+            fr = D.sinusoid_frequencies(W).to(dev)
+            toks = torch.randint(0, 32000, (T,), device=dev)
+            hbm("embed_sinusoid_prefill", _time_flushed(lambda: D.embed_sinusoid(toks, b.positions, tab, 3.0, fr)), T * W * 6)
+            hbm("tupidra_embed_prefill", _time_flushed(lambda: E.embed_scale(toks, tab, 1.0)), T * W * 8)
+            proj = torch.randn(T, aH * ad + Wc, device=dev).to(bf)
+            bytes_ = T * ((aH * ad + Wc) * 2 + aH * ad * 4 + Wc * 2)
+            t = _time_flushed(lambda: SA.window_kv_append(proj, None, aH, aG, ad, ae, False, 1e-6, b.slots, cache, qk_norm=True, q_temp=(0.1, 1024),
+                                                          positions=b.positions))
+            hbm("norm_temp_kv_append_prefill", t, bytes_)
+            bias = torch.randn(aH * ad + Wc, device=dev)
+            hbm("tupidra_kv_append_prefill", _time_flushed(lambda: SA.window_kv_append(proj, bias, aH, aG, ad, ae, True, 1e-6, b.slots, cache)), bytes_)
+            gu = torch.randn(T, 2 * F, device=dev).to(bf)
+            hbm("gated_clamped_prefill", _time_flushed(lambda: E.gated_clamped(gu, 7.0, 1.702)), T * F * 6)
+            hbm("gated_silu_prefill", _time_flushed(lambda: E.gated_silu(gu)), T * F * 6)
+    res.update(_gpt_kernels(dict(heads=aH, width=W, top=1, expert_ff=F), peaks))
+    res["native_launches"] = native.launch_count
+    return res
+
+
 def _gpt_kernels(size: Dict[str, Any], peaks: Dict[str, float]) -> Dict[str, Any]:
     """The GPT family's like kernels at like sizes: causal flash attention over the same 2 x 2048 tokens, paged decode
     attention over the same 32 contexts of 4096 (head size 128 for both), and the SwiGLU feed-forward's two GEMMs on
@@ -518,6 +666,9 @@ def run(which: str = "nafazen", sizes: List[str] | None = None, prompt_len: int 
     elif which == "tupidra":
         from ..models.tupidra import TupidraConfig as Config, example_config
         table, kernels = TUPIDRA_SIZES, _tupidra_kernels
+    elif which == "zokepel":
+        from ..models.zokepel import ZokepelConfig as Config, example_config
+        table, kernels = ZOKEPEL_SIZES, _zokepel_kernels
     else:
         raise ValueError(f"no architecture comparison for {which!r}")
     peaks = _peaks()
@@ -534,7 +685,7 @@ def run(which: str = "nafazen", sizes: List[str] | None = None, prompt_len: int 
         row = {"params": params, "gpt_params": gcfg.num_parameters(), "gpt_ffn": gcfg.ffn,
                which: _serve(ncfg, prompts, new_tokens, 64), "gpt": _serve(gcfg, prompts, new_tokens, 16),
                "kernels": kernels(size, peaks)}
-        if which == "tupidra" and name in NAMISUN_SIZES:          # the closest design: parallel layout, scans, state slots
+        if which in ("tupidra", "zokepel") and name in NAMISUN_SIZES:          # the closest design: parallel layout, scans, state slots
             from ..models.namisun import NamisunConfig, example_config as namisun_example
             ccfg = NamisunConfig.from_dict(namisun_example(**NAMISUN_SIZES[name]), name=f"namisun-{name}")
             row["namisun_params"] = ccfg.num_parameters()
