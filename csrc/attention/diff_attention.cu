@@ -627,7 +627,7 @@ static int launch_diff_attention_mma(const DiffAttnParams& p, int ntiles, int de
 #define LLMCTL_DM_LAUNCH(NT)                                                                                                     \
   do {                                                                                                                           \
     auto kern = diff_attention_mma_kernel<NT, SPLIT>;                                                                            \
-    if (smem > 48 * 1024) LLMCTL_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem))); \
+    if (smem > 46 * 1024) LLMCTL_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem))); \
     kern<<<grid, warps * 32, smem, s>>>(p, decode);                                                                              \
   } while (0)
   if (p.e <= 32) LLMCTL_DM_LAUNCH(4);
@@ -644,7 +644,7 @@ static int launch_diff_attention(const DiffAttnParams& p, int ntiles, size_t sme
 #define LLMCTL_DA_LAUNCH(NC)                                                                                                     \
   do {                                                                                                                           \
     auto kern = diff_attention_kernel<T, NC, SPLIT>;                                                                             \
-    if (smem > 48 * 1024) LLMCTL_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem))); \
+    if (smem > 46 * 1024) LLMCTL_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem))); \
     kern<<<grid, kDaThreads, smem, s>>>(p);                                                                                      \
   } while (0)
   if (p.e <= 32) LLMCTL_DA_LAUNCH(1);

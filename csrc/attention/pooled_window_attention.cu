@@ -348,7 +348,7 @@ LLMCTL_API int llmctl_window_qkv_write(const void* qkv, long long ld, const void
   cudaStream_t s = (cudaStream_t)stream;
   LLMCTL_DISPATCH_DTYPE(is_fp32, T, {
     auto kern = window_qkv_write_kernel<T>;
-    if (smem > 48 * 1024) LLMCTL_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
+    if (smem > 46 * 1024) LLMCTL_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
     kern<<<tokens, 256, smem, s>>>((const T*)qkv, ld, (const T*)bias, qn_w, kn_w, H, G, d, e, rot, freq, mult, eps, positions, slots,
                                    q_out, (T*)cache, bs, PS, (T*)v_first, v_mode, lam);
   });

@@ -693,7 +693,7 @@ static int launch_softcap_attention_mma(const SoftcapAttnParams& p, int ntiles, 
 #define LLMCTL_SW_LAUNCH(NT)                                                                                                     \
   do {                                                                                                                           \
     auto kern = softcap_attention_mma_kernel<NT, SPLIT>;                                                                         \
-    if (smem > 48 * 1024) LLMCTL_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem))); \
+    if (smem > 46 * 1024) LLMCTL_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem))); \
     kern<<<grid, warps * 32, smem, s>>>(p, decode);                                                                              \
   } while (0)
   if (p.e <= 32) LLMCTL_SW_LAUNCH(4);
@@ -710,7 +710,7 @@ static int launch_softcap_attention(const SoftcapAttnParams& p, int ntiles, size
 #define LLMCTL_SF_LAUNCH(NC)                                                                                                     \
   do {                                                                                                                           \
     auto kern = softcap_attention_kernel<T, NC, SPLIT>;                                                                          \
-    if (smem > 48 * 1024) LLMCTL_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem))); \
+    if (smem > 46 * 1024) LLMCTL_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem))); \
     kern<<<grid, kSwThreads, smem, s>>>(p);                                                                                      \
   } while (0)
   if (p.e <= 32) LLMCTL_SF_LAUNCH(1);

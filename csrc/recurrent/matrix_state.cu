@@ -860,7 +860,7 @@ static int launch_matrix_scan_cols(const MatrixScanParams& p, int nportions, cud
   constexpr int DP = RPT * LPC, COLS = 16 * CPL;
   const size_t smem = sizeof(float) * (2 * kMsTC * (static_cast<size_t>(DP) * (KIND == 0 ? 2 : 3) + COLS + 4) + 2 * kMsTC * COLS);
   auto kern = matrix_scan_kernel<RPT, LPC, CPL, KIND>;
-  if (smem > 48 * 1024) LLMCTL_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
+  if (smem > 46 * 1024) LLMCTL_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
   kern<<<dim3(nportions, p.H, (p.e + COLS - 1) / COLS), LPC * 16, smem, s>>>(p);
   return 0;
 }
@@ -888,7 +888,7 @@ template <typename T, int RPW, int KIND>
 static int launch_matrix_step(const MatrixStepParams& p, int nportions, cudaStream_t s) {
   const int vec = p.e % 4 == 0 ? 4 : 1;
   const size_t smem = sizeof(float) * (3 * RPW * 8 + 16 * 32 * static_cast<size_t>(vec) + 2 * static_cast<size_t>(p.e));
-  LLMCTL_REQUIRE(smem <= 48 * 1024);
+  LLMCTL_REQUIRE(smem <= 46 * 1024);
   const dim3 grid(nportions, p.G);
   if (vec == 4) matrix_step_kernel<T, RPW, 4, KIND><<<grid, 256, smem, s>>>(p);
   else matrix_step_kernel<T, RPW, 1, KIND><<<grid, 256, smem, s>>>(p);

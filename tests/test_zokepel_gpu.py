@@ -145,7 +145,8 @@ def test_bonus_memory_kernels(cuda_device, H, d):
 
 @pytest.mark.parametrize("H,G,d,e,n,bs,rows,far", [(4, 2, 8, 6, 45, 16, 8, 30.0), (3, 1, 5, 7, 133, 16, 4, 9.0), (8, 2, 16, 16, 300, 64, 16, 200.0),
                                                    (8, 4, 48, 40, 200, 64, 12, 17.5), (4, 4, 32, 64, 150, 8, 2, 3.0), (16, 2, 128, 128, 290, 64, 32, 128.0),
-                                                   (2, 1, 16, 136, 70, 16, 8, 64.0), (6, 6, 64, 72, 400, 64, 10, 600.0)])
+                                                   (2, 1, 16, 136, 70, 16, 8, 64.0), (6, 6, 64, 72, 400, 64, 10, 600.0),
+                                                   (2, 1, 64, 16, 140, 64, 6, 50.0)])      # shared memory exactly at the default limit
 def test_biased_attention_kernels(cuda_device, H, G, d, e, n, bs, rows, far):
     """Unit-RMS queries and keys with temperature, cache append and attention with a bias table on the FMA and tensor-core
     kernels: prompt tiles, single tokens, key slices; a prompt and a later portion of it."""
