@@ -41,18 +41,22 @@ CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-fvisibility=hidden", "-Wall", "-I",
 _SERVE_COMMON = ["common", "gemm", "activation", "moe", "comm/watchdog.cu"]    # the gated GEMM modes report expired flag waits through the watchdog
 COMPONENTS = {
     "serve": _SERVE_COMMON + ["norm", "rope", "swiglu", "serve", "attention/latent_attention.cu", "attention/latent_attention_t5.cu",
-                              "attention/pooled_window_attention.cu", "attention/pooled_window_attention_mma.cu",
+                              "attention/pooled_window_attention.cu", "attention/pooled_window_attention_mma.cu", "attention/qkv_write.cu",
                               "attention/diff_attention.cu", "attention/softcap_window_attention.cu", "recurrent"],
     # what trace replay of one design needs and no more (the library grows when another component is asked for later)
     "serve-nafazen": _SERVE_COMMON + ["norm/scalar_rmsnorm.cu", "attention/latent_attention.cu", "attention/latent_attention_t5.cu"],
     "serve-teluzen": _SERVE_COMMON + ["norm/sandwich_norm.cu", "attention/pooled_window_attention.cu",
-                                      "attention/pooled_window_attention_mma.cu"],
-    "serve-namisun": _SERVE_COMMON + ["norm/scalar_rmsnorm.cu", "norm/parallel_norm.cu", "attention/diff_attention.cu", "recurrent"],
+                                      "attention/pooled_window_attention_mma.cu", "attention/qkv_write.cu"],
+    "serve-namisun": _SERVE_COMMON + ["norm/scalar_rmsnorm.cu", "norm/parallel_norm.cu", "attention/diff_attention.cu", "recurrent/gla.cu",
+                                      "recurrent/selective_scan.cu"],
     "serve-tupidra": _SERVE_COMMON + ["norm/scalar_rmsnorm.cu", "norm/sandwich_norm.cu", "norm/canon_norm.cu",
                                       "attention/latent_attention.cu", "attention/latent_attention_t5.cu",
                                       "attention/softcap_window_attention.cu", "recurrent/selective_scan.cu"],
     "serve-zokepel": _SERVE_COMMON + ["norm/sandwich_norm.cu", "norm/dual_norm.cu", "attention/softcap_window_attention.cu",
                                       "recurrent/gla.cu", "recurrent/matrix_state.cu"],
+    "serve-kozasun": _SERVE_COMMON + ["norm/hyper_norm.cu", "attention/qkv_write.cu", "attention/softcap_window_attention.cu",
+                                      "attention/latent_attention.cu", "attention/latent_attention_t5.cu", "recurrent/gla.cu",
+                                      "recurrent/retention.cu"],
     "all": None,
 }
 

@@ -17,7 +17,10 @@
 //                             is loaded once for 16 tokens of a prompt portion (one head) or for 16 heads of a
 //                             decoded token.  Keys stream through shared memory in tiles of 32 with an online
 //                             softmax; the rotated query part is rotated on load.  Causal: a row at position p
-//                             sees cache positions 0..p of its sequence.  Long contexts are split over CTAs
+//                             sees cache positions 0..p of its sequence, or with `window` > 0 only the last `window`
+//                             of them (key tiles before the tile's first window are never read).  Optionally every
+//                             head's output is multiplied by sigmoid(head_gate[token, head]) (the value projection is
+//                             linear, so a gate per head may act before it).  Long contexts are split over CTAs
 //                             (`splits` > 1) and merged by a second kernel, as the decode kernel in
 //                             csrc/serve/paged_attention.cu does.  bf16 with R + dr a multiple of 16 runs both
 //                             products on the tensor cores (mma.sync m16n8k16, fp32 accumulation; softmax, masks
@@ -30,7 +33,7 @@
 namespace llmctl {
 
 // d: [tokens, ld] = [ q latent raw (Q) | kv latent raw (R) | key rope part raw (dr) ] (R = dr = 0 columns absent for
-// a layer that reads another layer's cache).
+// a layer that reads another layer's cache; Q = 0 for queries without a latent).
 template <typename T>
 __global__ void __launch_bounds__(128)
 latent_kv_write_kernel(const T* __restrict__ d, long long ld, int Q, int R, int dr, const T* __restrict__ wq,
@@ -40,14 +43,16 @@ latent_kv_write_kernel(const T* __restrict__ d, long long ld, int Q, int R, int 
   __shared__ float red[32];
   const long long tok = blockIdx.x;
   const T* row = d + tok * ld;
-  float ss = 0.f;
-  for (int c = threadIdx.x; c < Q; c += blockDim.x) {
-    const float v = to_f32(row[c]);
-    ss += v * v;
+  if (Q > 0) {
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < Q; c += blockDim.x) {
+      const float v = to_f32(row[c]);
+      ss += v * v;
+    }
+    ss = block_sum(ss, red);
+    const float rq = 1.f / sqrtf(ss / static_cast<float>(Q) + eps);
+    for (int c = threadIdx.x; c < Q; c += blockDim.x) cq[tok * Q + c] = from_f32<T>(to_f32(row[c]) * rq * to_f32(wq[c]));
   }
-  ss = block_sum(ss, red);
-  const float rq = 1.f / sqrtf(ss / static_cast<float>(Q) + eps);
-  for (int c = threadIdx.x; c < Q; c += blockDim.x) cq[tok * Q + c] = from_f32<T>(to_f32(row[c]) * rq * to_f32(wq[c]));
   if (R == 0) return;
   const long long slot = slots[tok];
   if (slot < 0) return;  // padded token: uniform over the block, nobody waits below
@@ -69,6 +74,18 @@ latent_kv_write_kernel(const T* __restrict__ d, long long ld, int Q, int R, int 
 constexpr int kRows = 16;      // query rows per CTA
 constexpr int kKeys = 32;      // keys per tile
 constexpr int kAttnThreads = 128;
+constexpr int kWindowAlign = 32;    // a window's first key tile starts at a multiple of this (a tcgen05 key tile never straddles a page)
+
+// First key that the tile whose first token is at position p_first reads.
+__device__ __forceinline__ int latent_first_key(int p_first, int window) {
+  return window > 0 ? max(p_first - window + 1, 0) / kWindowAlign * kWindowAlign : 0;
+}
+
+// Gate of a head's output: sigmoid of head_gate[token, head] (row stride gate_ld), 1 without one.
+template <typename T>
+__device__ __forceinline__ float latent_head_gate(const T* gate, long long gate_ld, long long tok, int h) {
+  return gate ? 1.f / (1.f + expf(-to_f32(gate[tok * gate_ld + h]))) : 1.f;
+}
 
 // tiles: int32 [ntiles, 4] = {first token row, token count, sequence row (block table), unused}
 // ql: fp32 [tokens, H, R] absorbed queries;  q: [tokens, ldq] raw queries, head h at h * (dn + dr), rope part last
@@ -79,7 +96,8 @@ latent_attention_kernel(const float* __restrict__ ql, long long ql_st, long long
                         const T* __restrict__ cache, const int* __restrict__ block_tables, int max_blocks,
                         int block_size, const int* __restrict__ tiles, const int* __restrict__ positions,
                         const float* __restrict__ freq, float mult, float scale, int H, int R, int dr, int heads_per_tile,
-                        int keys_per_split, T* __restrict__ out, float* __restrict__ partial, const float* __restrict__ sinks) {
+                        int keys_per_split, T* __restrict__ out, float* __restrict__ partial, const float* __restrict__ sinks,
+                        int window, const T* __restrict__ head_gate, long long gate_ld) {
   extern __shared__ float smem[];
   const int D = R + dr, Dp = D + 1;
   float* qs = smem;                      // [kRows][Dp]
@@ -129,7 +147,7 @@ latent_attention_kernel(const float* __restrict__ ql, long long ql_st, long long
     for (int i = 0; i < NC; ++i) acc[r][i] = 0.f;
 
   const int last = row_pos[nrows - 1];                     // positions grow with the token index
-  const int k_begin = split * keys_per_split;
+  const int k_begin = latent_first_key(row_pos[0], window) + split * keys_per_split;
   const int k_end = min(last + 1, k_begin + keys_per_split);
   for (int j0 = k_begin; j0 < k_end; j0 += kKeys) {
     __syncthreads();                                       // previous tile fully consumed (and qs written)
@@ -153,7 +171,7 @@ latent_attention_kernel(const float* __restrict__ ql, long long ql_st, long long
         float s = 0.f;
         for (int c = 0; c < D; ++c) s += qr[c] * kr[c];
         const int j = j0 + jj;
-        ps[r * kKeys + jj] = (j < k_end && j <= row_pos[r]) ? s : -INFINITY;
+        ps[r * kKeys + jj] = (j < k_end && j <= row_pos[r] && (window <= 0 || row_pos[r] - j < window)) ? s : -INFINITY;
       }
     }
     __syncthreads();
@@ -195,7 +213,7 @@ latent_attention_kernel(const float* __restrict__ ql, long long ql_st, long long
     const int tok = tok0 + r / nh, h = h0 + r % nh;
     const long long base = static_cast<long long>(tok) * H + h;
     if (nsplit == 1) {
-      const float inv = row_l[r] > 0.f ? 1.f / row_l[r] : 0.f;
+      const float inv = (row_l[r] > 0.f ? 1.f / row_l[r] : 0.f) * latent_head_gate(head_gate, gate_ld, tok, h);
 #pragma unroll
       for (int i = 0; i < NC; ++i) {
         const int c = tid + i * kAttnThreads;
@@ -218,7 +236,8 @@ latent_attention_kernel(const float* __restrict__ ql, long long ql_st, long long
 
 template <typename T>
 __global__ void __launch_bounds__(128)
-latent_attention_merge_kernel(const float* __restrict__ partial, T* __restrict__ out, int R, int nsplit) {
+latent_attention_merge_kernel(const float* __restrict__ partial, T* __restrict__ out, int R, int nsplit, int H,
+                              const T* __restrict__ head_gate, long long gate_ld) {
   const long long base = blockIdx.x;   // token * H + head
   const float* p = partial + base * nsplit * (R + 2);
   extern __shared__ float wsplit[];    // [nsplit]: exp(m_s - max m) / sum, 0 for empty splits
@@ -235,7 +254,7 @@ latent_attention_merge_kernel(const float* __restrict__ partial, T* __restrict__
     if (threadIdx.x == 0) {
       float gl = 0.f;
       for (int s = 0; s < nsplit; ++s) gl += p[s * (R + 2) + R + 1] * wsplit[s];
-      s_inv = gl > 0.f ? 1.f / gl : 0.f;
+      s_inv = (gl > 0.f ? 1.f / gl : 0.f) * latent_head_gate(head_gate, gate_ld, base / H, static_cast<int>(base % H));
     }
   }
   __syncthreads();
@@ -248,8 +267,10 @@ latent_attention_merge_kernel(const float* __restrict__ partial, T* __restrict__
 }
 
 // Used by the tcgen05 kernel's launcher (latent_attention_t5.cu) for split contexts.
-int launch_latent_attention_merge_bf16(const float* partial, void* out, int R, int splits, int rows, cudaStream_t s) {
-  latent_attention_merge_kernel<__nv_bfloat16><<<rows, 128, splits * sizeof(float), s>>>(partial, (__nv_bfloat16*)out, R, splits);
+int launch_latent_attention_merge_bf16(const float* partial, void* out, int R, int splits, int rows, int H, const void* head_gate,
+                                       long long gate_ld, cudaStream_t s) {
+  latent_attention_merge_kernel<__nv_bfloat16><<<rows, 128, splits * sizeof(float), s>>>(partial, (__nv_bfloat16*)out, R, splits, H,
+                                                                                         (const __nv_bfloat16*)head_gate, gate_ld);
   return 0;
 }
 
@@ -258,7 +279,7 @@ static int launch_latent_attention(const float* ql, long long ql_st, long long q
                                    const int* block_tables, int max_blocks, int block_size, const int* tiles, int ntiles,
                                    const int* positions, const float* freq, float mult, float scale, int H, int R, int dr,
                                    int heads_per_tile, int splits, int keys_per_split, void* out, float* partial,
-                                   int tokens, const float* sinks, cudaStream_t s) {
+                                   int tokens, const float* sinks, int window, const void* head_gate, long long gate_ld, cudaStream_t s) {
   const int D = R + dr;
   const size_t smem = (static_cast<size_t>(kRows + kKeys) * (D + 1) + kRows * kKeys + 4 * kRows) * sizeof(float);
   if (smem > 227 * 1024) return static_cast<int>(cudaErrorInvalidValue);
@@ -271,7 +292,7 @@ static int launch_latent_attention(const float* ql, long long ql_st, long long q
     if (e != cudaSuccess) return static_cast<int>(e);                                                                \
     kern<<<grid, kAttnThreads, smem, s>>>(ql, ql_st, ql_sh, (const T*)q, ldq, dn, (const T*)cache, block_tables, max_blocks, \
                                           block_size, tiles, positions, freq, mult, scale, H, R, dr, heads_per_tile, \
-                                          keys_per_split, (T*)out, partial, sinks);                                  \
+                                          keys_per_split, (T*)out, partial, sinks, window, (const T*)head_gate, gate_ld); \
   } while (0)
   if (nc <= 1) LAUNCH(1);
   else if (nc <= 2) LAUNCH(2);
@@ -280,7 +301,7 @@ static int launch_latent_attention(const float* ql, long long ql_st, long long q
   else return static_cast<int>(cudaErrorInvalidValue);
 #undef LAUNCH
   if (splits > 1)
-    latent_attention_merge_kernel<T><<<tokens * H, 128, splits * sizeof(float), s>>>(partial, (T*)out, R, splits);
+    latent_attention_merge_kernel<T><<<tokens * H, 128, splits * sizeof(float), s>>>(partial, (T*)out, R, splits, H, (const T*)head_gate, gate_ld);
   return 0;
 }
 
@@ -303,7 +324,7 @@ latent_attention_tc_kernel(const TQ* __restrict__ ql, long long ql_st, long long
                            int block_size, const int* __restrict__ tiles, const int* __restrict__ positions,
                            const float* __restrict__ freq, float mult, float scale, int H, int R, int dr, int heads_per_tile,
                            int keys_per_split, int stages, __nv_bfloat16* __restrict__ out, float* __restrict__ partial,
-                           const float* __restrict__ sinks) {
+                           const float* __restrict__ sinks, int window, const __nv_bfloat16* __restrict__ head_gate, long long gate_ld) {
   constexpr int kR = 16 * MT, kWarps = 8 * MT;
   extern __shared__ __align__(16) unsigned char smem_raw[];
   const int D = R + dr, Dp = D + 8;
@@ -356,7 +377,7 @@ latent_attention_tc_kernel(const TQ* __restrict__ ql, long long ql_st, long long
     for (int j = 0; j < 4; ++j) oacc[i][j] = 0.f;
 
   const int last = row_pos[nrows - 1];
-  const int k_begin = split * keys_per_split;
+  const int k_begin = latent_first_key(row_pos[0], window) + split * keys_per_split;
   const int k_end = min(last + 1, k_begin + keys_per_split);
   const int vec_per_row = D >> 3;
   // a warp per key row, asynchronous 16-byte copies of the cache rows as they are
@@ -414,7 +435,8 @@ latent_attention_tc_kernel(const TQ* __restrict__ ql, long long ql_st, long long
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int r = 16 * wm + g + (e >> 1) * 8, col = 8 * wn + 2 * t + (e & 1), j = j0 + col;
-        Ss[r * kSsLd + col] = (j < k_end && j <= row_pos[r]) ? (sacc[0][e] + sacc[1][e]) * scale : -INFINITY;
+        const bool seen = j < k_end && j <= row_pos[r] && (window <= 0 || row_pos[r] - j < window);
+        Ss[r * kSsLd + col] = seen ? (sacc[0][e] + sacc[1][e]) * scale : -INFINITY;
       }
     }
     __syncthreads();
@@ -469,7 +491,7 @@ latent_attention_tc_kernel(const TQ* __restrict__ ql, long long ql_st, long long
     if (r >= nrows) continue;
     const int tok = tok0 + r / nh, h = h0 + r % nh;
     const long long base = static_cast<long long>(tok) * H + h;
-    const float inv = row_l[r] > 0.f ? 1.f / row_l[r] : 0.f;
+    const float inv = (row_l[r] > 0.f ? 1.f / row_l[r] : 0.f) * (nsplit > 1 ? 1.f : latent_head_gate(head_gate, gate_ld, tok, h));
     float* dst = nsplit > 1 ? partial + (base * nsplit + split) * (R + 2) : nullptr;
 #pragma unroll
     for (int i = 0; i < NT; ++i) {
@@ -505,7 +527,8 @@ static int launch_latent_attention_tc(const TQ* ql, long long ql_st, long long q
                                       const int* block_tables, int max_blocks, int block_size, const int* tiles, int ntiles,
                                       const int* positions, const float* freq, float mult, float scale, int H, int R, int dr,
                                       int heads_per_tile, int splits, int keys_per_split, void* out, float* partial,
-                                      int tokens, int rows, const float* sinks, cudaStream_t s) {
+                                      int tokens, int rows, const float* sinks, int window, const void* head_gate, long long gate_ld,
+                                      cudaStream_t s) {
   // A second key-tile stage overlaps the copy of the next tile with the products of this one.  16-row tiles take it
   // only while two CTAs still share an SM (they overlap each other's copies anyway); 32-row tiles whenever it fits
   // (up to R + dr = 576 it does).
@@ -521,7 +544,8 @@ static int launch_latent_attention_tc(const TQ* ql, long long ql_st, long long q
     if (e != cudaSuccess) return static_cast<int>(e);                                                                \
     kern<<<grid, 256 * MT, smem, s>>>(ql, ql_st, ql_sh, (const __nv_bfloat16*)q, ldq, dn, (const __nv_bfloat16*)cache, \
                                       block_tables, max_blocks, block_size, tiles, positions, freq, mult, scale,     \
-                                      H, R, dr, heads_per_tile, keys_per_split, stages, (__nv_bfloat16*)out, partial, sinks); \
+                                      H, R, dr, heads_per_tile, keys_per_split, stages, (__nv_bfloat16*)out, partial, sinks, window, \
+                                      (const __nv_bfloat16*)head_gate, gate_ld); \
   } while (0)
 #define LAUNCH_TC_NT(MT)          \
   do {                            \
@@ -535,7 +559,8 @@ static int launch_latent_attention_tc(const TQ* ql, long long ql_st, long long q
 #undef LAUNCH_TC_NT
 #undef LAUNCH_TC
   if (splits > 1)
-    latent_attention_merge_kernel<__nv_bfloat16><<<tokens * H, 128, splits * sizeof(float), s>>>(partial, (__nv_bfloat16*)out, R, splits);
+    latent_attention_merge_kernel<__nv_bfloat16><<<tokens * H, 128, splits * sizeof(float), s>>>(partial, (__nv_bfloat16*)out, R, splits, H,
+                                                                                                 (const __nv_bfloat16*)head_gate, gate_ld);
   return 0;
 }
 
@@ -547,7 +572,7 @@ LLMCTL_API int llmctl_latent_kv_write(const void* d, long long ld, int Q, int R,
                                       void* cq, void* cache, const long long* slots, const int* positions,
                                       const float* freq, float mult, float eps, int tokens, int is_fp32, void* stream) {
   LLMCTL_BEGIN();
-  LLMCTL_REQUIRE(Q > 0 && R >= 0 && dr >= 0 && dr % 2 == 0 && ld >= Q + R + dr);
+  LLMCTL_REQUIRE(Q >= 0 && R >= 0 && Q + R > 0 && (Q == 0 || (wq != nullptr && cq != nullptr)) && dr >= 0 && dr % 2 == 0 && ld >= Q + R + dr);
   if (tokens == 0) return 0;
   LLMCTL_DISPATCH_DTYPE(is_fp32, T, (latent_kv_write_kernel<T><<<tokens, 128, 0, (cudaStream_t)stream>>>(
                                         (const T*)d, ld, Q, R, dr, (const T*)wq, (const T*)wkv, (T*)cq, (T*)cache, slots,
@@ -557,6 +582,8 @@ LLMCTL_API int llmctl_latent_kv_write(const void* d, long long ld, int Q, int R,
 
 // partial: fp32 scratch of tokens * H * splits * (R + 2) numbers when splits > 1 (may be null otherwise).
 // sinks: fp32 [H] or null; exp(sinks[h]) (not scaled) joins the softmax denominator of head h.
+// window: 0, or a row at position p sees p - window + 1 .. p (the keys of a slice are counted from the tile's first window, rounded
+// down to a multiple of 32).  head_gate: [tokens, H] in the activation type (row stride gate_ld) or null.
 // ql: absorbed queries, element (token, head, c) at ql[token * ql_st + head * ql_sh + c]; fp32, or bf16 (ql_bf16) on the
 // tensor-core path only (llmctl_latent_attention_uses_tensor_cores).
 LLMCTL_API int llmctl_latent_attention_uses_tensor_cores(int is_fp32, int R, int dr, int rows_per_tile) {
@@ -568,21 +595,23 @@ LLMCTL_API int llmctl_latent_attention(const void* ql, int ql_bf16, long long ql
                                        int ntiles, int tokens, const int* positions, const float* freq, float mult,
                                        float scale, int H, int R, int dr, int heads_per_tile, int splits,
                                        int keys_per_split, void* out, float* partial, int is_fp32, int tensor_cores,
-                                       int rows_per_tile, const float* sinks, void* stream) {
+                                       int rows_per_tile, const float* sinks, int window, const void* head_gate, long long gate_ld,
+                                       void* stream) {
   LLMCTL_BEGIN();
   LLMCTL_REQUIRE(H > 0 && R > 0 && dr >= 0 && dr % 2 == 0 && block_size > 0 && heads_per_tile >= 1 &&
-                 heads_per_tile <= rows_per_tile && (rows_per_tile == 16 || rows_per_tile == 32) && splits >= 1 && keys_per_split > 0 && (splits == 1 || partial != nullptr));
+                 heads_per_tile <= rows_per_tile && (rows_per_tile == 16 || rows_per_tile == 32) && splits >= 1 && keys_per_split > 0 && (splits == 1 || partial != nullptr) && window >= 0);
   if (ntiles == 0) return 0;
   int rc;
   if (!is_fp32 && tensor_cores && latent_attention_tc_ok(R, dr, rows_per_tile) && keys_per_split % kTcKeys == 0) {
     if (ql_bf16)
       rc = launch_latent_attention_tc<__nv_bfloat16>((const __nv_bfloat16*)ql, ql_st, ql_sh, q, ldq, dn, cache, block_tables, max_blocks,
                                                      block_size, tiles, ntiles, positions, freq, mult, scale, H, R, dr, heads_per_tile,
-                                                     splits, keys_per_split, out, partial, tokens, rows_per_tile, sinks, (cudaStream_t)stream);
+                                                     splits, keys_per_split, out, partial, tokens, rows_per_tile, sinks, window, head_gate, gate_ld,
+                                                     (cudaStream_t)stream);
     else
     rc = launch_latent_attention_tc<float>((const float*)ql, ql_st, ql_sh, q, ldq, dn, cache, block_tables, max_blocks, block_size, tiles, ntiles, positions, freq,
                                     mult, scale, H, R, dr, heads_per_tile, splits, keys_per_split, out, partial, tokens,
-                                    rows_per_tile, sinks, (cudaStream_t)stream);
+                                    rows_per_tile, sinks, window, head_gate, gate_ld, (cudaStream_t)stream);
     if (rc != 0) LLMCTL_FAIL(rc, "latent attention launch");
     LLMCTL_RETURN_LAST();
   }
@@ -590,7 +619,7 @@ LLMCTL_API int llmctl_latent_attention(const void* ql, int ql_bf16, long long ql
   LLMCTL_DISPATCH_DTYPE(is_fp32, T, (rc = launch_latent_attention<T>((const float*)ql, ql_st, ql_sh, q, ldq, dn, cache, block_tables, max_blocks, block_size,
                                                                      tiles, ntiles, positions, freq, mult, scale, H, R, dr,
                                                                      heads_per_tile, splits, keys_per_split, out, partial,
-                                                                     tokens, sinks, (cudaStream_t)stream)));
+                                                                     tokens, sinks, window, head_gate, gate_ld, (cudaStream_t)stream)));
   if (rc != 0) LLMCTL_FAIL(rc, "latent attention launch");
   LLMCTL_RETURN_LAST();
 }

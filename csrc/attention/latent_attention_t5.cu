@@ -2,12 +2,15 @@
 //
 //   out[t, h, :] = softmax_j( scale * q[t, h, :] . k[j, :] ) c[j, :]      k[j] = [c[j] | kr[j]]  (one cache row, D = R + dr)
 //
+// over the keys 0 .. t of the sequence or, with a window, its last `window` ones (tiles before a CTA's first window are not read);
+// optionally times sigmoid(head_gate[t, h]).
+//
 // A CTA owns 128 (token, head) query rows — 128 tokens of one head in batches with prompt portions, one token's heads
 // when every sequence decodes — and one group of up to 256 output columns (the fp32 accumulator of 128 x R would fill
 // tensor memory on its own at R = 512, so the columns are split over CTAs and each recomputes the scores).
 //
-//   * queries: assembled once per call as [tokens, heads, D] bf16 (absorbed part | rotated rope part), one TMA tile
-//     of 128 x D per CTA (128-byte swizzle, D / 64 panels)
+//   * queries: assembled once per call as [tokens, heads, D] bf16 (absorbed part | rotated rope part), or without a rope part
+//     read as the projection left them ([heads, tokens, R]); one TMA tile of 128 x D per CTA (128-byte swizzle, D / 64 panels)
 //   * keys: tiles of 32 cache rows fetched by TMA straight from the paged cache through the block table (a tile never
 //     straddles a page: the page size is a multiple of 32), double-buffered; the same tile is the K-major B operand of
 //     S = Q K^T (UMMA 128 x 32 x 16 over D) and, through its first R columns, the MN-major B operand of O += P C
@@ -82,7 +85,8 @@ latent_attention_t5_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
                            const int* __restrict__ block_tables, int max_blocks, int block_size,
                            const int* __restrict__ tiles, const int* __restrict__ positions, float scale, int H, int R,
                            int dr, int heads_per_tile, int keys_per_split, int nsplit, int q_rows_are_heads,
-                           __nv_bfloat16* __restrict__ out, float* __restrict__ partial, const float* __restrict__ sinks) {
+                           __nv_bfloat16* __restrict__ out, float* __restrict__ partial, const float* __restrict__ sinks, int window,
+                           const __nv_bfloat16* __restrict__ head_gate, long long gate_ld, int q_head_rows) {
   using namespace t5;
   extern __shared__ uint8_t smem_raw[];
   __shared__ uint64_t bar_q, bar_kfull[2], bar_kempty[2], bar_s[2], bar_p, bar_pv;
@@ -103,7 +107,8 @@ latent_attention_t5_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
   const int cg = blockIdx.z % ncg, split = blockIdx.z / ncg;
   const int col0 = cg * kColGroup, ncols = min(kColGroup, R - col0);
   const int* bt = block_tables + static_cast<long long>(seq) * max_blocks;
-  const int k_begin = split * keys_per_split;
+  const int k_first = window > 0 ? max(positions[tok0] - window + 1, 0) / kKeys * kKeys : 0;      // whole key tiles
+  const int k_begin = k_first + split * keys_per_split;
   const int k_end = min(positions[tok0 + ntok - 1] + 1, k_begin + keys_per_split);
   const int ntile = k_end > k_begin ? (k_end - k_begin + kKeys - 1) / kKeys : 0;
 
@@ -154,8 +159,9 @@ latent_attention_t5_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
     // ------------------------------ TMA producer ------------------------------
     if (lane == 0) {
       mbar_expect_tx(&bar_q, q_bytes);
-      const int qcol0 = q_rows_are_heads ? 0 : h0 * D;
-      const int qrow0 = q_rows_are_heads ? tok0 * H + h0 : tok0;
+      // q_head_rows > 0: queries lie as [heads, q_head_rows tokens, D]; rows past the tile's tokens are never stored
+      const int qcol0 = (q_rows_are_heads || q_head_rows) ? 0 : h0 * D;
+      const int qrow0 = q_rows_are_heads ? tok0 * H + h0 : q_head_rows ? h0 * q_head_rows + tok0 : tok0;
       for (int p = 0; p < panels; ++p) tma_load_2d(smem + p * kQPanel, &tmQ, &bar_q, qcol0 + 64 * p, qrow0);
       int issued = 0;
       auto slot_of = [&](int i) {
@@ -264,13 +270,15 @@ latent_attention_t5_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
       uint32_t r[32];
       tmem_ld_x32(tS, r);
       tmem_ld_wait();
-      const int vis = min(pos, k_end - 1) - (k_begin + kKeys * i) + 1;      // the first `vis` keys of the tile are visible
+      // keys lo .. vis - 1 of the tile are visible
+      const int vis = min(pos, k_end - 1) - (k_begin + kKeys * i) + 1;
+      const int lo = window > 0 ? pos - window + 1 - (k_begin + kKeys * i) : 0;
       float bm = -INFINITY;
 #pragma unroll
       for (int e = 0; e < 32; ++e) {
         const float v = __uint_as_float(r[e]) * scale_log2;
         r[e] = __float_as_uint(v);
-        if (e < vis) bm = fmaxf(bm, v);
+        if (e < vis && e >= lo) bm = fmaxf(bm, v);
       }
       // lazy reference: move it only when the tile's maximum outgrows it by more than 2^8
       const bool need = bm > m_ref + kRescaleThreshold;
@@ -284,8 +292,8 @@ latent_attention_t5_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
       uint32_t pk[16];
 #pragma unroll
       for (int e = 0; e < 32; e += 2) {
-        const float p0 = e < vis ? exp2f(__uint_as_float(r[e]) + neg) : 0.f;
-        const float p1 = e + 1 < vis ? exp2f(__uint_as_float(r[e + 1]) + neg) : 0.f;
+        const float p0 = (e < vis && e >= lo) ? exp2f(__uint_as_float(r[e]) + neg) : 0.f;
+        const float p1 = (e + 1 < vis && e + 1 >= lo) ? exp2f(__uint_as_float(r[e + 1]) + neg) : 0.f;
         l += p0 + p1;
         pk[e >> 1] = pack_bf16x2(p0, p1);
       }
@@ -317,7 +325,8 @@ latent_attention_t5_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
     }
     if (ok) {
       const long long base = static_cast<long long>(tok) * H + h;
-      const float inv = l > 0.f ? 1.f / l : 0.f;
+      float inv = l > 0.f ? 1.f / l : 0.f;
+      if (head_gate && valid) inv *= 1.f / (1.f + expf(-__bfloat162float(head_gate[tok * gate_ld + h])));
       float* pdst = partial != nullptr ? partial + (base * nsplit + split) * (R + 2) : nullptr;
 #pragma unroll 1
       for (int c = 0; c < ncols; c += 32) {
@@ -356,7 +365,8 @@ latent_attention_t5_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
 }
 
 // defined in latent_attention.cu: out[row, :] = sum over splits of the partial sums, renormalised
-int launch_latent_attention_merge_bf16(const float* partial, void* out, int R, int splits, int rows, cudaStream_t s);
+int launch_latent_attention_merge_bf16(const float* partial, void* out, int R, int splits, int rows, int H, const void* head_gate,
+                                       long long gate_ld, cudaStream_t s);
 
 }  // namespace llmctl
 
@@ -384,21 +394,27 @@ LLMCTL_API int llmctl_latent_attention_t5_status(int clear) {
 // tiles: int32 [ntiles, 4] = (first token row, tokens, block-table row, 0); a tile holds tokens x heads_per_tile <= 128
 // query rows, and more than one head per tile only with single-token tiles.  qfull: bf16 scratch [tokens, H, R + dr].
 // cache_rows: rows of the cache tensor (blocks x block_size).  partial: fp32 [tokens * H * splits * (R + 2)] when
-// splits > 1.  ql as in llmctl_latent_attention.
+// splits > 1.  ql, window, head_gate as in llmctl_latent_attention.  qfull may be null when dr is 0 and ql is bf16, contiguous as
+// [heads, tokens, R] and 16-byte aligned, with one head per tile: the queries are then read where they are.
 LLMCTL_API int llmctl_latent_attention_t5(const void* ql, int ql_bf16, long long ql_st, long long ql_sh, const void* q,
                                           long long ldq, int dn, const void* cache, long long cache_rows,
                                           const int* block_tables, int max_blocks, int block_size, const int* tiles,
                                           int ntiles, int tokens, const int* positions, const float* freq, float mult,
                                           float scale, int H, int R, int dr, int heads_per_tile, int splits,
-                                          int keys_per_split, void* qfull, void* out, float* partial, const float* sinks, void* stream) {
+                                          int keys_per_split, void* qfull, void* out, float* partial, const float* sinks, int window,
+                                          const void* head_gate, long long gate_ld, void* stream) {
   LLMCTL_BEGIN();
   LLMCTL_REQUIRE(llmctl_latent_attention_t5_ok(R, dr, block_size) && H > 0 && heads_per_tile >= 1 &&
                  heads_per_tile <= t5::kRows && splits >= 1 && keys_per_split > 0 && keys_per_split % t5::kKeys == 0 &&
-                 (splits == 1 || partial != nullptr) && qfull != nullptr && cache_rows >= block_size);
+                 (splits == 1 || partial != nullptr) && cache_rows >= block_size && window >= 0);
+  LLMCTL_REQUIRE(qfull != nullptr || (dr == 0 && ql_bf16 && heads_per_tile == 1 && ql_st == R && ql_sh == static_cast<long long>(tokens) * R &&
+                                      (reinterpret_cast<uintptr_t>(ql) & 15) == 0));
   if (ntiles == 0 || tokens == 0) return 0;
   cudaStream_t s = (cudaStream_t)stream;
   const int D = R + dr;
-  if (ql_bf16)
+  if (qfull == nullptr) {
+    // nothing to assemble
+  } else if (ql_bf16)
     latent_q_assemble_kernel<__nv_bfloat16><<<tokens * H, 128, 0, s>>>((const __nv_bfloat16*)ql, ql_st, ql_sh, (const __nv_bfloat16*)q,
                                                                         ldq, dn, positions, freq, mult, H, R, dr, (__nv_bfloat16*)qfull);
   else
@@ -406,7 +422,8 @@ LLMCTL_API int llmctl_latent_attention_t5(const void* ql, int ql_bf16, long long
                                                                 positions, freq, mult, H, R, dr, (__nv_bfloat16*)qfull);
   const int rows_are_heads = heads_per_tile > 1 ? 1 : 0;
   CUtensorMap tmQ, tmK;
-  int rc = rows_are_heads ? get_tmap_2d_bf16(&tmQ, qfull, static_cast<uint64_t>(tokens) * H, D, D, t5::kRows, 64, 1)
+  int rc = qfull == nullptr ? get_tmap_2d_bf16(&tmQ, ql, static_cast<uint64_t>(tokens) * H, D, D, t5::kRows, 64, 1)
+         : rows_are_heads ? get_tmap_2d_bf16(&tmQ, qfull, static_cast<uint64_t>(tokens) * H, D, D, t5::kRows, 64, 1)
                           : get_tmap_2d_bf16(&tmQ, qfull, tokens, static_cast<uint64_t>(H) * D, static_cast<uint64_t>(H) * D, t5::kRows, 64, 1);
   if (rc) LLMCTL_FAIL(rc, "tensor map Q");
   rc = get_tmap_2d_bf16(&tmK, cache, cache_rows, D, D, t5::kKeys, 64, 1);
@@ -417,9 +434,10 @@ LLMCTL_API int llmctl_latent_attention_t5(const void* ql, int ql_bf16, long long
   dim3 grid(ntiles, (H + heads_per_tile - 1) / heads_per_tile, splits * ncg);
   latent_attention_t5_kernel<<<grid, t5::kThreads, smem, s>>>(tmQ, tmK, block_tables, max_blocks, block_size, tiles, positions,
                                                                scale, H, R, dr, heads_per_tile, keys_per_split, splits,
-                                                               rows_are_heads, (__nv_bfloat16*)out, splits > 1 ? partial : nullptr, sinks);
+                                                               rows_are_heads, (__nv_bfloat16*)out, splits > 1 ? partial : nullptr, sinks, window,
+                                                               (const __nv_bfloat16*)head_gate, gate_ld, qfull == nullptr ? tokens : 0);
   if (splits > 1) {
-    rc = launch_latent_attention_merge_bf16(partial, out, R, splits, tokens * H, s);
+    rc = launch_latent_attention_merge_bf16(partial, out, R, splits, tokens * H, H, head_gate, gate_ld, s);
     if (rc) LLMCTL_FAIL(rc, "merge");
   }
   LLMCTL_RETURN_LAST();

@@ -10,10 +10,7 @@
 // all heads]); rows bs.. are the pooled rows of the blocks whose first token lies in the page (PS = ceil(bs / P) of
 // them at most), so pooled rows are owned, freed and reused with the page.
 //
-//   llmctl_window_qkv_write : per token, from the packed projection [q | k | v]: + bias, RMS norm over the whole q
-//       and the whole k projection (per-coordinate weights), rotation of the first `rot` numbers of every head as
-//       interleaved pairs at the token's position, value mixing v <- (1-lam) v + lam v_first with the values an
-//       earlier layer computed for the same token; q leaves in fp32, k and v go to the token's cache row.
+//   (llmctl_window_qkv_write, which fills the token rows, is in csrc/attention/qkv_write.cu)
 //   llmctl_window_pool_update : for every token of the step that completes a block, the block's pooled row.
 //   llmctl_pooled_window_attention : scores * scale * temp[h] in fp32, softmax over the visible tokens and blocks,
 //       optional mixing of the NORMALISED weights across heads (w'_h = sum_g talk[h,g] w_g), then w' V with the
@@ -26,69 +23,9 @@
 #include <limits.h>
 
 #include "../common/dtype.cuh"
-#include "../rope/rope_interleaved.cuh"
 #include "pooled_window.cuh"
 
 namespace llmctl {
-
-// ---------------------------------------------------------------------------------------------------------------
-// projection post-processing + cache append: one CTA per token
-// ---------------------------------------------------------------------------------------------------------------
-template <typename T>
-__global__ void __launch_bounds__(256)
-window_qkv_write_kernel(const T* __restrict__ qkv, long long ld, const T* __restrict__ bias, const float* __restrict__ qn_w,
-                        const float* __restrict__ kn_w, int H, int G, int d, int e, int rot, const float* __restrict__ freq,
-                        float mult, float eps, const int* __restrict__ positions, const long long* __restrict__ slots,
-                        float* __restrict__ q_out, T* __restrict__ cache, int bs, int PS, T* __restrict__ v_first, int v_mode,
-                        const float* __restrict__ lam) {
-  extern __shared__ float buf[];      // [H*d + G*d]
-  __shared__ float red[32];
-  const long long t = blockIdx.x;
-  const int Nq = H * d, Nk = G * d, Nv = G * e, Wc = Nk + Nv;
-  const T* row = qkv + t * ld;
-  float* sq = buf;
-  float* sk = buf + Nq;
-  float ssq = 0.f, ssk = 0.f;
-  for (int c = threadIdx.x; c < Nq + Nk; c += blockDim.x) {
-    float v = to_f32(row[c]);
-    if (bias) v += to_f32(bias[c]);
-    buf[c] = v;
-    if (c < Nq) ssq += v * v;
-    else ssk += v * v;
-  }
-  ssq = block_sum(ssq, red);
-  ssk = block_sum(ssk, red);
-  const float rq = qn_w ? 1.f / sqrtf(ssq / static_cast<float>(Nq) + eps) : 1.f;
-  const float rk = kn_w ? 1.f / sqrtf(ssk / static_cast<float>(Nk) + eps) : 1.f;
-  for (int c = threadIdx.x; c < Nq + Nk; c += blockDim.x) {
-    if (c < Nq) sq[c] = sq[c] * rq * (qn_w ? qn_w[c] : 1.f);
-    else sk[c - Nq] = sk[c - Nq] * rk * (kn_w ? kn_w[c - Nq] : 1.f);
-  }
-  __syncthreads();
-  const int pos = positions[t];
-  const long long slot = slots[t];
-  T* crow = slot >= 0 ? cache + ((slot / bs) * (bs + PS) + slot % bs) * Wc : nullptr;
-  for (int c = threadIdx.x; c < Nq + Nk; c += blockDim.x) {
-    const bool isq = c < Nq;
-    const int cc = isq ? c : c - Nq;
-    const float* src = isq ? sq : sk;
-    const int dd = cc % d, base = cc - dd;
-    float v = src[cc];
-    if (dd < rot) v = rope_interleaved_coord([&](int k) { return src[base + k]; }, dd, pos, freq, mult);
-    if (isq) q_out[t * Nq + cc] = v;
-    else if (crow) crow[cc] = from_f32<T>(v);
-  }
-  const float l = (v_mode == 2) ? lam[0] : 0.f;
-  for (int c = threadIdx.x; c < Nv; c += blockDim.x) {
-    float v = to_f32(row[Nq + Nk + c]);
-    if (bias) v += to_f32(bias[Nq + Nk + c]);
-    const T vt = from_f32<T>(v);               // the projection's output in the activation type
-    if (v_mode == 1) v_first[t * Nv + c] = vt;
-    v = to_f32(vt);
-    if (v_mode == 2) v = (1.f - l) * v + l * to_f32(v_first[t * Nv + c]);
-    if (crow) crow[Nk + c] = from_f32<T>(v);
-  }
-}
 
 // one CTA per token; only the tokens that end a block do anything
 template <typename T>
@@ -329,31 +266,6 @@ static cudaError_t pwa_launch(const PwaParams& p, int ntiles, size_t smem, cudaS
 }  // namespace llmctl
 
 using namespace llmctl;
-
-// qkv: [tokens, H*d + G*d + G*e] (row stride ld) in the activation type; bias: same width or null; qn_w / kn_w: fp32
-// norm weights over the whole q / k projection, or null for no norm; rot: rotated numbers per head (even, <= d), freq:
-// fp32 [rot/2]; q_out: fp32 [tokens, H*d]; cache: [pages, bs + PS, G*(d+e)]; slots: int64 [tokens] = page * bs + offset
-// (negative: the token is not cached); v_mode: 0 plain, 1 also store the values in v_first [tokens, G*e], 2 mix with
-// v_first by lam (one fp32 number on the device).
-LLMCTL_API int llmctl_window_qkv_write(const void* qkv, long long ld, const void* bias, const float* qn_w, const float* kn_w,
-                                       int H, int G, int d, int e, int rot, const float* freq, float mult, float eps,
-                                       const int* positions, const long long* slots, float* q_out, void* cache, int bs, int PS,
-                                       void* v_first, int v_mode, const float* lam, int tokens, int is_fp32, void* stream) {
-  LLMCTL_BEGIN();
-  LLMCTL_REQUIRE(H > 0 && G > 0 && H % G == 0 && d > 0 && e > 0 && rot >= 0 && rot <= d && rot % 2 == 0 && bs > 0 && PS >= 0);
-  LLMCTL_REQUIRE(v_mode == 0 || (v_first != nullptr && (v_mode == 1 || lam != nullptr)));
-  if (tokens == 0) return 0;
-  const size_t smem = static_cast<size_t>(H + G) * d * sizeof(float);
-  LLMCTL_REQUIRE(smem <= 200 * 1024);
-  cudaStream_t s = (cudaStream_t)stream;
-  LLMCTL_DISPATCH_DTYPE(is_fp32, T, {
-    auto kern = window_qkv_write_kernel<T>;
-    if (smem > 46 * 1024) LLMCTL_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
-    kern<<<tokens, 256, smem, s>>>((const T*)qkv, ld, (const T*)bias, qn_w, kn_w, H, G, d, e, rot, freq, mult, eps, positions, slots,
-                                   q_out, (T*)cache, bs, PS, (T*)v_first, v_mode, lam);
-  });
-  LLMCTL_RETURN_LAST();
-}
 
 // seq_rows: int32 [tokens] = block-table row of each token's sequence; Wc = G*(d+e).
 LLMCTL_API int llmctl_window_pool_update(void* cache, const int* positions, const long long* slots, const int* seq_rows,

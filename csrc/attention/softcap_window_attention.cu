@@ -3,7 +3,7 @@
 //
 // H query heads use G key/value heads (head h reads head h / (H/G)).  For query position i and key position j <= i:
 //
-//     visible(i, j) = window == 0  or  i - j < window  or  j < keep_first
+//     visible(i, j) = j >= first(i)  or  j < keep_first,   first(i) = max(window > 0: i - window + 1,  chunk > 0: i - i mod chunk, 0)
 //     s_ij = q_i . k_j * scale;   cap > 0:  s_ij <- cap * tanh(s_ij / cap);   s_ij <- s_ij - slope_h * (i - j)
 //     p_ij = exp(s_ij) / (sum_visible exp(s_ij') + exp(sink_h))            sinks == null: no sink term
 //     o_i  = sum_j p_ij v_j,  times sigmoid(gate[i, h, :]) where a gate is given
@@ -110,7 +110,7 @@ struct SoftcapAttnParams {
   const float* table;        // [H, table_len] bias by distance, or null
   int table_len;
   float scale, cap;
-  int window, keep_first;
+  int window, keep_first, chunk;
   int H, G, d, e, bs;
   int HB;                    // heads per CTA
   void* out;                 // [T, H*e]
@@ -119,14 +119,21 @@ struct SoftcapAttnParams {
   float* part_o;             // [tiles * H/HB * splits, 32, e]
 };
 
+// First key of the window / chunk of a query at position i (kept first tokens aside); never falls as i grows.
+__device__ __forceinline__ int sw_first_key(int i, const SoftcapAttnParams& p) {
+  int lo = p.window > 0 ? max(i - p.window + 1, 0) : 0;
+  if (p.chunk > 0) lo = max(lo, i - i % p.chunk);
+  return lo;
+}
+
 // The key tiles of a query tile whose positions are p_first .. p_last: tiles 0 .. nA-1 cover the kept first tokens
 // [0, endA), tiles nA .. nA+nB-1 the window [wb, p_last + 1).
 struct KeyTiles {
   int endA, wb, nkeys, nA, nB;
-  __device__ KeyTiles(int p_first, int p_last, int window, int keep_first) {
+  __device__ KeyTiles(int p_first, int p_last, const SoftcapAttnParams& p) {
     nkeys = p_last + 1;
-    wb = window > 0 ? max(p_first - window + 1, 0) : 0;
-    endA = window > 0 ? min(keep_first, wb) : 0;
+    wb = sw_first_key(p_first, p);
+    endA = min(p.keep_first, wb);
     nA = (endA + kSwKT - 1) / kSwKT;
     nB = (nkeys - wb + kSwKT - 1) / kSwKT;
   }
@@ -134,8 +141,8 @@ struct KeyTiles {
   __device__ int limit(int it) const { return it < nA ? endA : nkeys; }
 };
 
-__device__ __forceinline__ bool sw_visible(int qpos, int key, int window, int keep_first) {
-  return key <= qpos && (window <= 0 || qpos - key < window || key < keep_first);
+__device__ __forceinline__ bool sw_visible(int qpos, int first, int key, int keep_first) {
+  return key <= qpos && (key >= first || key < keep_first);
 }
 
 // NC: output columns per lane (e <= 32 * NC)
@@ -169,12 +176,13 @@ softcap_attention_kernel(const SoftcapAttnParams p) {
 
   float m[4], l[4], acc[4][NC], slope[4];
   const float* tab[4];
-  int qpos[4];
+  int qpos[4], qlo[4];
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
     const int r = warp * 4 + i;
     const int h = h0 + (r < nrows ? r % HB : 0);
     qpos[i] = r < nrows ? p_first + r / HB : -1;
+    qlo[i] = sw_first_key(max(qpos[i], 0), p);
     slope[i] = p.slopes ? p.slopes[h] : 0.f;
     tab[i] = p.table ? p.table + static_cast<long long>(h) * p.table_len : nullptr;
     const bool sink = p.sinks != nullptr && split == 0;
@@ -185,7 +193,7 @@ softcap_attention_kernel(const SoftcapAttnParams p) {
   }
   const int warp_rows = min(max(nrows - warp * 4, 0), 4);
 
-  const KeyTiles kt(p_first, p_last, p.window, p.keep_first);
+  const KeyTiles kt(p_first, p_last, p);
   int it_begin = 0, it_end = kt.nA + kt.nB;
   if (SPLIT) {
     const int per = (it_end + p.splits - 1) / p.splits;
@@ -236,7 +244,7 @@ softcap_attention_kernel(const SoftcapAttnParams p) {
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         if (i < warp_rows) {
-          const bool seen = lane < nk && sw_visible(qpos[i], j, p.window, p.keep_first);
+          const bool seen = lane < nk && sw_visible(qpos[i], qlo[i], j, p.keep_first);
           float sv = -INFINITY;
           if (seen) {
             sv = p.cap > 0.f ? p.cap * tanhf(s[i] / p.cap) : s[i];
@@ -421,7 +429,7 @@ softcap_attention_mma_kernel(const SoftcapAttnParams p, int decode) {
     }
   }
 
-  const KeyTiles kt(p_first, p_last, p.window, p.keep_first);
+  const KeyTiles kt(p_first, p_last, p);
   int it_begin = 0, it_end = kt.nA + kt.nB;
   if (SPLIT) {
     const int per = (it_end + p.splits - 1) / p.splits;
@@ -465,7 +473,8 @@ softcap_attention_mma_kernel(const SoftcapAttnParams p, int decode) {
   // keys this warp's rows can see: the kept first tokens and [warp_wb, warp_last]
   const int warp_first = decode ? p_first : p_first + warp * 16;
   const int warp_last = decode ? p_first : p_first + min(warp * 16 + 15, nvalid - 1);
-  const int warp_wb = p.window > 0 ? warp_first - p.window + 1 : 0;
+  const int warp_wb = sw_first_key(warp_first, p);
+  const int qfirst_lo = sw_first_key(max(qpos_lo, 0), p), qfirst_hi = sw_first_key(max(qpos_hi, 0), p);
 
   float O[NT][4];
   float mrow[2], lrow[2];                 // lo / hi row; maxima in units of ln 2
@@ -543,8 +552,8 @@ softcap_attention_mma_kernel(const SoftcapAttnParams p, int decode) {
         }
         s_lo *= kSwLog2e;
         s_hi *= kSwLog2e;
-        S[nt][j] = (in && sw_visible(qpos_lo, key, p.window, p.keep_first)) ? s_lo : -INFINITY;
-        S[nt][2 + j] = (in && sw_visible(qpos_hi, key, p.window, p.keep_first)) ? s_hi : -INFINITY;
+        S[nt][j] = (in && sw_visible(qpos_lo, qfirst_lo, key, p.keep_first)) ? s_lo : -INFINITY;
+        S[nt][2 + j] = (in && sw_visible(qpos_hi, qfirst_hi, key, p.keep_first)) ? s_hi : -INFINITY;
         mx_lo = fmaxf(mx_lo, S[nt][j]);
         mx_hi = fmaxf(mx_hi, S[nt][2 + j]);
       }
@@ -724,21 +733,21 @@ static int launch_softcap_attention(const SoftcapAttnParams& p, int ntiles, size
 
 // tile_tokens: most tokens in a tile (<= 16; the tensor-core kernel, use_mma, takes 1 or up to 128); splits > 1 needs
 // part_ml [ntiles * H/HB * splits * 64] and part_o [ntiles * H/HB * splits * 32 * e] (fp32) and, on the tensor-core
-// kernel, tile_tokens 1.  window 0: every earlier key is seen.  cap 0: no soft cap.
+// kernel, tile_tokens 1.  window 0 and chunk 0: every earlier key is seen.  cap 0: no soft cap.
 // table: fp32 [H, table_len] or null.
 LLMCTL_API int llmctl_softcap_window_attention(const float* q, const void* cache, const int* block_tables, int max_blocks,
                                                const int* tiles, int ntiles, int tile_tokens, const int* positions, const void* gate,
                                                long long gate_ld, const float* slopes, const float* sinks, const float* table, int table_len,
-                                               float scale, float cap, int window, int keep_first, int H, int G, int d, int e, int bs, void* out, int splits,
+                                               float scale, float cap, int window, int keep_first, int chunk, int H, int G, int d, int e, int bs, void* out, int splits,
                                                float* part_ml, float* part_o, int is_fp32, int use_mma, void* stream) {
   LLMCTL_BEGIN();
   LLMCTL_REQUIRE(H > 0 && G > 0 && H % G == 0 && d > 0 && e > 0 && e <= 512 && bs > 0 && tile_tokens >= 1 && window >= 0 &&
-                 keep_first >= 0 && cap >= 0.f);
+                 keep_first >= 0 && chunk >= 0 && cap >= 0.f);
   LLMCTL_REQUIRE(table == nullptr || table_len >= 1);
   LLMCTL_REQUIRE(splits >= 1 && (splits == 1 || (part_ml != nullptr && part_o != nullptr)));
   if (ntiles == 0) return 0;
   cudaStream_t s = (cudaStream_t)stream;
-  SoftcapAttnParams p{q, cache, block_tables, max_blocks, tiles, positions, gate, gate_ld, slopes, sinks, table, table_len, scale, cap, window, keep_first,
+  SoftcapAttnParams p{q, cache, block_tables, max_blocks, tiles, positions, gate, gate_ld, slopes, sinks, table, table_len, scale, cap, window, keep_first, chunk,
                       H, G, d, e, bs, llmctl_softcap_attention_heads_per_cta(H, G, tile_tokens, use_mma), out, splits, part_ml, part_o};
   LLMCTL_REQUIRE(p.HB >= 1);
   const int head_blocks = H / p.HB;

@@ -6,8 +6,9 @@
 //                        (ties: lowest index), optionally renormalised to sum 1; optional per-token gate
 //                        sigmoid(wg . x) of a shared expert; counts tokens per expert.  Optionally the CHOICE is made on
 //                        score + correction[e] (the weights stay the plain scores) and restricted to the
-//                        `keep_groups` of `n_groups` equal groups of neighbouring experts whose best choice score is
-//                        largest (the others count as minus infinity).  Expert ids >= the number of experts with
+//                        `keep_groups` of `n_groups` equal groups of neighbouring experts whose group score is largest
+//                        (the others count as minus infinity); a group's score is its best choice score or the sum of
+//                        its two best.  The weights may be multiplied by a constant.  Expert ids >= the number of experts with
 //                        weights (`E` of plan / permute) are identity experts: they get no rows in the permuted
 //                        buffer and the combine adds weight * (the token's input) for them.
 //   llmctl_moe_plan    : one CTA: per-expert row offsets in the permuted buffer, every expert's segment padded to a
@@ -36,7 +37,7 @@ template <typename T>
 __global__ void __launch_bounds__(256)
 moe_route_kernel(const float* __restrict__ x, const T* __restrict__ wr, const T* __restrict__ wg, int W, int E, int top,
                  int softmax_scores, int renormalise, const float* __restrict__ correction, int n_groups, int keep_groups,
-                 int* __restrict__ ids, float* __restrict__ weights, float* __restrict__ gate, int* __restrict__ counts) {
+                 int group_best, float weight_scale, int* __restrict__ ids, float* __restrict__ weights, float* __restrict__ gate, int* __restrict__ counts) {
   extern __shared__ float score[];   // [E] scores, then [E] choice scores
   float* choice = score + E;
   const long long tok = blockIdx.x;
@@ -76,7 +77,7 @@ moe_route_kernel(const float* __restrict__ x, const T* __restrict__ wr, const T*
     }
     for (int e = 0; e < E; ++e) choice[e] = score[e] + (correction ? correction[e] : 0.f);
     if (n_groups > 1 && keep_groups < n_groups) {
-      // a group's score is its largest choice score; groups outside the best `keep_groups` cannot be chosen
+      // a group's score is its largest choice score, or the sum of its two largest; groups outside the best `keep_groups` cannot be chosen
       const int gs = E / n_groups;
       unsigned long long kept = 0ull;                  // n_groups <= 64
       for (int r = 0; r < keep_groups; ++r) {
@@ -84,8 +85,12 @@ moe_route_kernel(const float* __restrict__ x, const T* __restrict__ wr, const T*
         float bgv = -INFINITY;
         for (int gi = 0; gi < n_groups; ++gi) {
           if (kept >> gi & 1ull) continue;
-          float gv = -INFINITY;
-          for (int e = gi * gs; e < (gi + 1) * gs; ++e) gv = fmaxf(gv, choice[e]);
+          float gv = -INFINITY, second = -INFINITY;
+          for (int e = gi * gs; e < (gi + 1) * gs; ++e) {
+            second = fmaxf(second, fminf(gv, choice[e]));
+            gv = fmaxf(gv, choice[e]);
+          }
+          if (group_best == 2 && gs > 1) gv += second;
           if (bg < 0 || gv > bgv) {
             bgv = gv;
             bg = gi;
@@ -125,6 +130,8 @@ moe_route_kernel(const float* __restrict__ x, const T* __restrict__ wr, const T*
       for (int k = 0; k < top; ++k) weights[tok * top + k] /= z;
     } else if (renormalise)
       for (int k = 0; k < top; ++k) weights[tok * top + k] /= total + 1e-20f;
+    if (weight_scale != 1.f)
+      for (int k = 0; k < top; ++k) weights[tok * top + k] *= weight_scale;
   }
 }
 
@@ -311,17 +318,17 @@ LLMCTL_API int llmctl_moe_tile_rows() { return kTileM; }
 
 LLMCTL_API int llmctl_moe_route(const float* x, const void* wr, const void* wg, int is_fp32, int tokens, int W, int E, int top,
                                 int softmax_scores, int renormalise, const float* correction, int n_groups, int keep_groups,
-                                int* ids, float* weights, float* gate, int* counts, void* stream) {
+                                int group_best, float weight_scale, int* ids, float* weights, float* gate, int* counts, void* stream) {
   LLMCTL_BEGIN();
   LLMCTL_REQUIRE(E >= 1 && top >= 1 && top <= E && E <= 4096 && (wg == nullptr || gate != nullptr));
   LLMCTL_REQUIRE(n_groups <= 1 || (n_groups <= 64 && E % n_groups == 0 && keep_groups >= 1 && keep_groups <= n_groups &&
-                                   keep_groups * (E / n_groups) >= top));
+                                   keep_groups * (E / n_groups) >= top && (group_best == 1 || group_best == 2)));
   cudaStream_t s = (cudaStream_t)stream;
   LLMCTL_CHECK(cudaMemsetAsync(counts, 0, sizeof(int) * E, s));
   if (tokens == 0) return 0;
   LLMCTL_DISPATCH_DTYPE(is_fp32, T, (moe_route_kernel<T><<<tokens, 256, 2 * E * sizeof(float), s>>>(
                                         x, (const T*)wr, (const T*)wg, W, E, top, softmax_scores, renormalise, correction, n_groups,
-                                        keep_groups, ids, weights, gate, counts)));
+                                        keep_groups, group_best, weight_scale, ids, weights, gate, counts)));
   LLMCTL_RETURN_LAST();
 }
 

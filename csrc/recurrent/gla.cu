@@ -190,7 +190,7 @@ gla_output_kernel(const float* __restrict__ o, const float* __restrict__ w, int 
   const float f = 1.f / sqrtf(ss / e + eps);
   for (int c = lane; c < e; c += 32) {
     const float g = to_f32(gate[t * ldg + h * e + c]);
-    out[r * e + c] = from_f32<T>(orow[c] * f * w[h * w_stride + c] * ((gate_sigmoid ? 1.f : g) / (1.f + expf(-g))));
+    out[r * e + c] = from_f32<T>(orow[c] * f * (w ? w[h * w_stride + c] : 1.f) * ((gate_sigmoid ? 1.f : g) / (1.f + expf(-g))));
   }
 }
 
@@ -222,7 +222,7 @@ LLMCTL_API int llmctl_gla_scan(const void* q, long long ldq, const void* k, long
   LLMCTL_RETURN_LAST();
 }
 
-// o: fp32 [T, H * e]; w: fp32 [e] (w_stride 0) or [H, e] (w_stride e); gate: [T, H * e] (row stride ldg) pre-activation;
+// o: fp32 [T, H * e]; w: fp32 [e] (w_stride 0) or [H, e] (w_stride e), or null (no weight); gate: [T, H * e] (row stride ldg) pre-activation;
 // out: [T, H * e] in the activation type.
 LLMCTL_API int llmctl_gla_output(const float* o, const float* w, int w_stride, const void* gate, long long ldg, int gate_sigmoid, void* out,
                                  int tokens, int H, int e, float eps, int is_fp32, void* stream) {

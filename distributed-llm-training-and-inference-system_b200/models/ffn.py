@@ -98,18 +98,19 @@ class GatedExpertMoE(nn.Module):
     when ``shared_gate``.  Optional parts: ``identity`` further router outputs behind the experts stand for identity
     experts (output = input, no weights); ``correction``: a learned vector added to the scores for the choice only;
     ``groups`` = (count, keep): the router outputs form ``count`` equal groups of neighbours and only the ``keep`` groups
-    with the largest best choice score can be chosen from; ``clamp`` = (limit, alpha): the experts compute
+    with the largest group score can be chosen from, the sum of a group's ``group_best`` (1 or 2) largest choice scores;
+    ``weight_scale``: a constant on the routing weights; ``clamp`` = (limit, alpha): the experts compute
     ``g sigmoid(alpha g) (u + 1)`` on ``g = min(gate, limit)``, ``u = clamp(up, -limit, limit)`` instead of the gated
     SiLU."""
 
     def __init__(self, width: int, experts: int, top: int, ff: int, shared_ff: Optional[int], dtype, device, *,
                  scale_input: bool = True, softmax_scores: bool = False, renormalise: bool = False, shared_gate: bool = True,
                  identity: int = 0, correction: bool = False, groups: Optional[Tuple[int, int]] = None,
-                 clamp: Optional[Tuple[float, float]] = None):
+                 clamp: Optional[Tuple[float, float]] = None, group_best: int = 1, weight_scale: float = 1.0):
         super().__init__()
         kw = dict(dtype=dtype, device=device)
         self.top, self.scale_input, self.softmax_scores, self.renormalise = top, scale_input, softmax_scores, renormalise
-        self.groups, self.clamp = groups, clamp
+        self.groups, self.clamp, self.group_best, self.weight_scale = groups, clamp, group_best, weight_scale
         if groups and ((experts + identity) % groups[0] or not 1 <= groups[1] <= groups[0] or groups[1] * ((experts + identity) // groups[0]) < top):
             raise ValueError(f"expert groups {groups} do not fit {experts} + {identity} router outputs with {top} choices")
         self.router = nn.Parameter(torch.empty(experts + identity, width, **kw))
@@ -146,4 +147,5 @@ class GatedExpertMoE(nn.Module):
             shared = ops.linear(eops.gated_silu(ops.linear(h, self.shared_gate_up)), self.shared_down)
         return mops.moe_ffn(x32, h.dtype, self.router, self.gate_up, self.down, self.top, scale_input=self.scale_input,
                             shared_out=shared, w_shared_gate=self.shared_gate, softmax=self.softmax_scores,
-                            renormalise=self.renormalise, correction=self.correction, groups=self.groups, clamp=self.clamp)
+                            renormalise=self.renormalise, correction=self.correction, groups=self.groups, clamp=self.clamp,
+                            group_best=self.group_best, weight_scale=self.weight_scale)

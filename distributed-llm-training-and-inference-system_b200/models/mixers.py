@@ -14,16 +14,22 @@ single rotated key part shared by all heads.  Queries go through their own norme
 
 Optional parts of ``LatentAttention`` (fields of its spec): ``sink`` — a learned number per head whose exponential joins
 the softmax denominator (a key without a value, not scaled); ``out_gate`` — the concatenated heads are multiplied element
-by element with the sigmoid of one more projection of the mixer's input (packed into the down-projection GEMM).
+by element with the sigmoid of one more projection of the mixer's input (packed into the down-projection GEMM);
+``head_gate`` — the same with one number per head, applied by the attention kernel; ``window`` — a token sees itself and the
+``window - 1`` tokens before it.  ``q_rank`` 0: queries are projected from the mixer's input directly (in the same packed
+GEMM), ``rot_dim`` 0: no rotated part.
 
-``SoftcapWindowAttention``: grouped-query attention without rotation whose scores pass a tanh soft cap and lose a linear
-distance bias with one slope per head; a sliding window that also keeps the first tokens of the sequence; a softmax with
-one added to the denominator (a sink of score 0); values cached at unit RMS per head; projection biases; a sigmoid output
+``SoftcapWindowAttention``: grouped-query attention whose scores pass a tanh soft cap and lose a linear
+distance bias with one slope per head; a sliding window that also keeps the first tokens of the sequence; chunks (a query
+sees the keys of its own chunk only); a softmax with one added to the denominator (a sink of score 0) or with a learned
+sink per head; an RMS norm over the whole q and k projections and rotation of the first ``rot_dims`` numbers of every head
+(pairs (i, i + rot_dims/2)); values cached at unit RMS per head; projection biases; a sigmoid output
 gate; queries and keys at unit RMS per head; a query temperature that grows with the position; a learned bias per
 logarithmic distance bucket.  Every part is a field of ``SoftcapWindowAttentionSpec``.  Per step:
 
     p        = h Wp^T                           (one packed GEMM: q | k | v | gate)
-    q, cache = bias / value norm / append       (ops.softcap_attention.window_kv_append)
+    q, cache = bias / value norm / append       (ops.softcap_attention.window_kv_append, or with projection norms or
+                                                 rotation ops.window_attention.window_qkv_write)
     o        = attention over kept + window keys, gate      (ops.softcap_attention.softcap_window_attention)
     out      = o Wo^T + bo
 
@@ -73,6 +79,10 @@ both low-rank projections, ``ops.matrix_state.delta_rule``, the output GEMM.
 and a silu gate.  Per step: ``ops.matrix_state.token_shift``, one batched GEMM (r, k, v, gate), the low-rank decay (two GEMMs and
 a tanh), ``ops.matrix_state.bonus_memory``, the output GEMM.
 
+``Retention``: ``S <- decay_h S + k v^T,  o = S^T q`` with a fixed decay per head on rotated queries and keys; heads brought to
+unit RMS and gated by silu of a projection.  Per step: one packed GEMM (q | k | v | gate), ``ops.retention.retention``, the
+output GEMM.
+
 ``BranchPair``: two mixers side by side on one input; its output is an ``ops.dual_norm.BranchSum`` that the residual update
 evaluates (each branch RMS-normed over the model width with a weight of its own, half their sum).
 
@@ -91,10 +101,15 @@ from ..ops import functional as ops
 from ..ops import latent_attention as lops
 from ..ops import matrix_state as mops
 from ..ops import recurrent as rops
+from ..ops import retention as retops
 from ..ops import softcap_attention as sops
 from ..ops import window_attention as wops
 from ..ops.dual_norm import BranchSum
 from ..ops.elementwise import rope_frequencies, sigmoid_gate_, tanh_
+
+
+def _pad8(n: int) -> int:
+    return (n + 7) // 8 * 8
 
 
 @dataclass
@@ -111,6 +126,8 @@ class LatentAttentionSpec:
     kv_from: Optional[int] = None       # index of the layer whose cache this layer reads
     sink: bool = False                  # a learned number per head joins the softmax denominator
     out_gate: bool = False              # heads * sigmoid(Wg h) before the output projection
+    head_gate: bool = False             # the same with one gate per head
+    window: int = 0                     # a token sees itself and the window - 1 tokens before it; 0: every earlier token
 
     @property
     def cache_width(self) -> int:
@@ -125,14 +142,21 @@ class LatentAttention(nn.Module):
         s = self.spec = spec
         self.eps = eps
         own = s.kv_from is None
+        if (s.out_gate and s.head_gate) or s.window < 0 or (s.q_rank == 0 and not own):
+            raise ValueError(f"inconsistent latent attention parts: {s}")
         kw = dict(dtype=dtype, device=device)
         self.n_down = s.q_rank + (s.kv_rank + s.rot_dim if own else 0)
-        rows = self.n_down + (s.heads * s.vdim if s.out_gate else 0)
-        self.w_down = nn.Parameter(torch.empty(rows, width, **kw))                      # [dq ; dkv ; gate]
+        # rows of the packed projection: [dq ; dkv ; gate], or without a query latent [dkv ; q ; gate], those parts starting at
+        # multiples of 8
+        self.q_at = 0 if s.q_rank else _pad8(self.n_down)
+        self.gate_at = self.n_down if s.q_rank else self.q_at + _pad8(s.heads * (s.dim + s.rot_dim))
+        n_gate = s.heads * s.vdim if s.out_gate else s.heads if s.head_gate else 0
+        rows = self.gate_at + n_gate
+        self.w_down = nn.Parameter(torch.zeros(rows if s.q_rank else _pad8(rows), width, **kw))
         self.sink = nn.Parameter(torch.zeros(s.heads, dtype=torch.float32, device=device)) if s.sink else None
-        self.q_norm = nn.Parameter(torch.ones(s.q_rank, **kw))
+        self.q_norm = nn.Parameter(torch.ones(s.q_rank, **kw)) if s.q_rank else None
         self.kv_norm = nn.Parameter(torch.ones(s.kv_rank, **kw)) if own else None
-        self.w_uq = nn.Parameter(torch.empty(s.heads * (s.dim + s.rot_dim), s.q_rank, **kw))
+        self.w_uq = nn.Parameter(torch.empty(s.heads * (s.dim + s.rot_dim), s.q_rank, **kw)) if s.q_rank else None
         self.w_uk = nn.Parameter(torch.empty(s.heads, s.dim, s.kv_rank, **kw))          # per head [dn, R]
         self.w_uv = nn.Parameter(torch.empty(s.heads, s.vdim, s.kv_rank, **kw))         # per head [dv, R]
         self.w_o = nn.Parameter(torch.empty(width, s.heads * s.vdim, **kw))
@@ -142,14 +166,17 @@ class LatentAttention(nn.Module):
     def load(self, get, prefix: str) -> None:
         s = self.spec
         with torch.no_grad():
-            parts = [get(prefix + "dq")] + ([get(prefix + "dkv")] if s.kv_from is None else []) + ([get(prefix + "g")] if s.out_gate else [])
-            self.w_down.copy_(torch.cat(parts, dim=0))
+            parts = ([(0, "dq")] if s.q_rank else [(self.q_at, "q")]) + ([(s.q_rank, "dkv")] if s.kv_from is None else [])
+            for at, name in parts + ([(self.gate_at, "g")] if s.out_gate or s.head_gate else []):
+                w = get(prefix + name)
+                self.w_down[at:at + w.shape[0]].copy_(w)
             if s.sink:
                 self.sink.copy_(get(prefix + "sink").float())
-            self.q_norm.copy_(get(prefix + "dq.norm"))
+            if s.q_rank:
+                self.q_norm.copy_(get(prefix + "dq.norm"))
+                self.w_uq.copy_(get(prefix + "uq"))
             if s.kv_from is None:
                 self.kv_norm.copy_(get(prefix + "dkv.norm"))
-            self.w_uq.copy_(get(prefix + "uq"))
             self.w_uk.copy_(get(prefix + "uk").view(s.heads, s.dim, s.kv_rank))
             self.w_uv.copy_(get(prefix + "uv").view(s.heads, s.vdim, s.kv_rank))
             self.w_o.copy_(get(prefix + "o"))
@@ -162,8 +189,9 @@ class LatentAttention(nn.Module):
         d = ops.linear(h, self.w_down)
         cq = lops.latent_kv_write(d, s.q_rank, s.kv_rank if own else 0, s.rot_dim if own else 0, self.q_norm, self.kv_norm,
                                   cache if own else None, batch.slots, batch.positions, self.rot_freq, self.rot_mult, self.eps)
-        q = ops.linear(cq, self.w_uq)                                                   # [T, H * (dn + dr)]
-        qn = q.view(T, s.heads, s.dim + s.rot_dim)[:, :, :s.dim].transpose(0, 1)        # [H, T, dn], a view
+        nq = s.heads * (s.dim + s.rot_dim)
+        q = ops.linear(cq, self.w_uq) if s.q_rank else d[:, self.q_at:self.q_at + nq]   # [T, H * (dn + dr)]
+        qn = q.unflatten(1, (s.heads, s.dim + s.rot_dim))[:, :, :s.dim].transpose(0, 1) # [H, T, dn], a view
         # absorbed queries ql[t, h] = Uk_h^T qn[t, h]: fp32, except that the tensor-core attention kernel takes them
         # in bf16 (it multiplies in bf16 anyway); the kernel reads the [H, T, R] product through its strides
         if q.is_cuda and q.dtype == torch.bfloat16:
@@ -180,12 +208,15 @@ class LatentAttention(nn.Module):
             rows = lops.ROWS_PER_TILE_TCGEN05
         else:
             rows = lops.rows_per_tile(q.dtype, s.kv_rank, s.rot_dim, q.is_cuda, s.heads if batch.decode_only else lops.ROWS_PER_TILE_WIDE)
+        hpt = batch.heads_per_tile(s.heads, rows)
+        span = lops.key_span(batch.max_context, s.window, rows // hpt)
         ol = lops.latent_attention(ql, q, s.dim, cache, batch.block_tables, batch.tiles(rows), batch.positions,
-                                   self.rot_freq, self.rot_mult, s.scale, batch.heads_per_tile(s.heads, rows), batch.max_context,
-                                   batch.attention_splits(s.heads, rows), rows=rows, sinks=self.sink)
+                                   self.rot_freq, self.rot_mult, s.scale, hpt, batch.max_context,
+                                   batch.attention_splits(s.heads, rows, span), rows=rows, sinks=self.sink, window=s.window,
+                                   head_gate=d[:, self.gate_at:self.gate_at + s.heads] if s.head_gate else None)
         o = torch.bmm(ol.transpose(0, 1), self.w_uv.transpose(1, 2)).transpose(0, 1).reshape(T, s.heads * s.vdim)
         if s.out_gate:
-            o = sigmoid_gate_(o, d[:, self.n_down:])
+            o = sigmoid_gate_(o, d[:, self.gate_at:self.gate_at + s.heads * s.vdim])
         return ops.linear(o, self.w_o)
 
     def cache_shape(self, num_blocks: int, block_size: int) -> Tuple[int, ...]:
@@ -306,6 +337,12 @@ class SoftcapWindowAttentionSpec:
     q_temp: Optional[Tuple[float, float]] = None    # (coef, every): q *= 1 + coef ln(floor((p + 1) / every) + 1)
     bias_rows: int = 0          # rows of a learned bias per distance bucket and head (0: none)
     bias_max: float = 0.0       # distance at which the last bucket begins at the latest
+    chunk: int = 0              # position i sees only keys of its own chunk of this many positions; 0: no chunks
+    sink: bool = False          # a learned number per head joins the softmax denominator (instead of sink_one)
+    proj_norm: bool = False     # RMS norm over the whole q and the whole k projection, per-coordinate weights
+    rot_dims: int = 0           # rotated numbers per head, pairs (i, i + rot_dims/2); 0: no rotation
+    rot_base: float = 10000.0
+    out_bias: bool = True       # with ``bias``: the output projection has one too
 
     @property
     def cache_width(self) -> int:
@@ -318,8 +355,12 @@ class SoftcapWindowAttention(nn.Module):
     def __init__(self, width: int, spec: SoftcapWindowAttentionSpec, eps: float, dtype, device):
         super().__init__()
         s = self.spec = spec
-        if s.heads % s.kv_heads or s.window < 0 or s.keep_first < 0 or s.softcap < 0:
+        if s.heads % s.kv_heads or s.window < 0 or s.keep_first < 0 or s.softcap < 0 or s.chunk < 0 or (s.sink and s.sink_one):
             raise ValueError(f"inconsistent attention sizes: {s}")
+        # projection norms and rotation come with their own append kernel, which has no per-head norms and no temperature
+        self.rotary_append = s.proj_norm or s.rot_dims > 0
+        if self.rotary_append and (s.value_norm or s.qk_norm or s.q_temp or s.rot_dims % 2 or s.rot_dims > s.dim):
+            raise ValueError(f"attention parts that do not go together: {s}")
         self.eps = eps
         kw = dict(dtype=dtype, device=device)
         f32 = dict(dtype=torch.float32, device=device)
@@ -328,9 +369,15 @@ class SoftcapWindowAttention(nn.Module):
         self.w_in = nn.Parameter(torch.empty(self.n_qkv + (s.heads * s.vdim if s.out_gate else 0), width, **kw))     # [q ; k ; v ; gate]
         self.b_in = nn.Parameter(torch.zeros(self.n_qkv, **f32)) if s.bias else None
         self.w_o = nn.Parameter(torch.empty(width, s.heads * s.vdim, **kw))
-        self.b_o = nn.Parameter(torch.zeros(width, **f32)) if s.bias else None
+        self.b_o = nn.Parameter(torch.zeros(width, **f32)) if s.bias and s.out_bias else None
+        self.q_norm = nn.Parameter(torch.ones(self.nq, **f32)) if s.proj_norm else None
+        self.k_norm = nn.Parameter(torch.ones(self.nk, **f32)) if s.proj_norm else None
+        self.register_buffer("rot_freq", rope_frequencies(s.rot_dims, s.rot_base)[0].to(device) if s.rot_dims else None, persistent=False)
         self.register_buffer("slopes", sops.distance_slopes(s.heads).to(device) if s.distance_bias else None, persistent=False)
-        self.register_buffer("sinks", torch.zeros(s.heads, **f32) if s.sink_one else None, persistent=False)
+        if s.sink:
+            self.sinks = nn.Parameter(torch.zeros(s.heads, **f32))
+        else:
+            self.register_buffer("sinks", torch.zeros(s.heads, **f32) if s.sink_one else None, persistent=False)
         self.rel = nn.Parameter(torch.zeros(s.bias_rows, s.heads, **f32)) if s.bias_rows else None
         self._table: Optional[torch.Tensor] = None          # the learned bias by distance, formed on first use
 
@@ -340,7 +387,7 @@ class SoftcapWindowAttention(nn.Module):
         return self._table
 
     def load(self, get, prefix: str) -> None:
-        """Checkpoint names under ``prefix``: q, k, v (+ ``.b`` biases), g, rel ([rows, heads]), o (+ ``o.b``)."""
+        """Checkpoint names under ``prefix``: q, k, v (+ ``.b`` biases), q.norm, k.norm, sink, g, rel ([rows, heads]), o (+ ``o.b``)."""
         s = self.spec
         with torch.no_grad():
             parts = [get(prefix + "q"), get(prefix + "k"), get(prefix + "v")] + ([get(prefix + "g")] if s.out_gate else [])
@@ -348,7 +395,13 @@ class SoftcapWindowAttention(nn.Module):
             self.w_o.copy_(get(prefix + "o"))
             if s.bias:
                 self.b_in.copy_(torch.cat([get(prefix + "q.b"), get(prefix + "k.b"), get(prefix + "v.b")], dim=0).float())
+            if self.b_o is not None:
                 self.b_o.copy_(get(prefix + "o.b").float())
+            if s.proj_norm:
+                self.q_norm.copy_(get(prefix + "q.norm").float())
+                self.k_norm.copy_(get(prefix + "k.norm").float())
+            if s.sink:
+                self.sinks.copy_(get(prefix + "sink").float())
             if self.rel is not None:
                 self.rel.copy_(get(prefix + "rel").float())
         self._table = None
@@ -360,15 +413,19 @@ class SoftcapWindowAttention(nn.Module):
         """h: [T, W] in the activation type; ``cache``: this layer's [pages, bs, G (d + e)]."""
         s = self.spec
         p = ops.linear(h, self.w_in)
-        q = sops.window_kv_append(p, self.b_in, s.heads, s.kv_heads, s.dim, s.vdim, s.value_norm, self.eps, batch.slots, cache,
-                                  qk_norm=s.qk_norm, q_temp=s.q_temp, positions=batch.positions)
+        if self.rotary_append:
+            q = wops.window_qkv_write(p, self.b_in, self.q_norm, self.k_norm, s.heads, s.kv_heads, s.dim, s.vdim, s.rot_dims, self.rot_freq, 1.0,
+                                      self.eps, batch.positions, batch.slots, cache, batch.block_size, rot_half=True)
+        else:
+            q = sops.window_kv_append(p, self.b_in, s.heads, s.kv_heads, s.dim, s.vdim, s.value_norm, self.eps, batch.slots, cache,
+                                      qk_norm=s.qk_norm, q_temp=s.q_temp, positions=batch.positions)
         gate = p[:, self.n_qkv:] if s.out_gate else None
         # prompt portions: tiles of 128 tokens on the tensor-core kernel, of 16 on the FMA kernel; decoded tokens: one each
         width = sops.tile_width(cache.dtype, s.heads, s.kv_heads, s.dim, s.vdim, q.is_cuda, batch.decode_only)
         o = sops.softcap_window_attention(q, cache, batch.block_tables, batch.tiles(width), 1 if batch.decode_only else width,
                                           batch.positions, gate, self.slopes, self.sinks, s.scale, s.softcap, s.window, s.keep_first,
                                           s.heads, s.kv_heads, s.dim, s.vdim, batch.block_size, h.dtype, max_context=batch.max_context,
-                                          table=self.bias_table())
+                                          table=self.bias_table(), chunk=s.chunk)
         y = ops.linear(o, self.w_o)
         return y if self.b_o is None else torch.add(y, self.b_o)        # fp32 sum: the residual update takes either type
 
@@ -561,10 +618,6 @@ class SelectiveScan(nn.Module):
         return ops.linear(y, self.w_o)
 
 
-def _pad8(n: int) -> int:
-    return (n + 7) // 8 * 8
-
-
 @dataclass
 class DeltaRuleSpec:
     heads: int
@@ -715,6 +768,60 @@ class BonusMemory(nn.Module):
         z = ops.linear(tanh_(ops.linear(mix[4], self.w_1)), self.w_2)
         y = mops.bonus_memory(r, k, v, z, self.w_0, self.u, g, self.norm, h, batch.portions, state[0], state[1], s.heads, s.dim, self.eps,
                               decode=batch.decode_only)
+        return ops.linear(y, self.w_o)
+
+
+@dataclass
+class RetentionSpec:
+    heads: int
+    dim: int            # query / key size per head
+    vdim: int           # value size per head
+    decay: Tuple[float, ...]    # one per head
+    rot_dims: int = 0   # rotated numbers per head, pairs (i, i + rot_dims/2); 0: no rotation
+    rot_base: float = 10000.0
+
+
+class Retention(nn.Module):
+    stateful = True
+
+    def __init__(self, width: int, spec: RetentionSpec, eps: float, dtype, device):
+        super().__init__()
+        s = self.spec = spec
+        if len(s.decay) != s.heads or s.dim > retops.MAX_DIM or s.rot_dims % 2 or s.rot_dims > s.dim:
+            raise ValueError(f"inconsistent retention sizes: {s}")
+        self.eps = eps
+        nk, nv = s.heads * s.dim, s.heads * s.vdim
+        self.at: Dict[str, Tuple[int, int]] = {}         # columns of the packed projection, parts starting at multiples of 8
+        rows = 0
+        for name, n in (("q", nk), ("k", nk), ("v", nv), ("g", nv)):
+            self.at[name] = (rows, rows + n)
+            rows += _pad8(n)
+        self.w_in = nn.Parameter(torch.zeros(rows, width, dtype=dtype, device=device))
+        self.w_o = nn.Parameter(torch.empty(width, nv, dtype=dtype, device=device))
+        freq = rope_frequencies(s.rot_dims, s.rot_base)[0] if s.rot_dims else torch.zeros(1)
+        self.register_buffer("rot_freq", freq.to(device), persistent=False)
+        decay_m1 = torch.tensor([float(g) - 1.0 for g in s.decay], dtype=torch.float64).to(torch.float32)
+        self.register_buffer("decay_m1", decay_m1.to(device), persistent=False)
+
+    def load(self, get, prefix: str) -> None:
+        """Checkpoint names under ``prefix``: q, k, v, g, o."""
+        with torch.no_grad():
+            self.w_in.zero_()
+            for name, (a, b) in self.at.items():
+                self.w_in[a:b].copy_(get(prefix + name))
+            self.w_o.copy_(get(prefix + "o"))
+
+    def state_shapes(self) -> Tuple[Tuple[int, ...], ...]:
+        s = self.spec
+        return ((s.heads, s.dim, s.vdim),)
+
+    def forward(self, h: torch.Tensor, batch, state) -> torch.Tensor:
+        """h: [T, W] in the activation type; ``state``: (this layer run's [slots, H, d, e] fp32,)."""
+        s = self.spec
+        p = ops.linear(h, self.w_in)
+        q, k, v, g = (p[:, a:b] for a, b in self.at.values())
+        y = retops.retention(q, k, v, g, batch.positions, self.rot_freq, s.rot_dims, self.decay_m1, batch.portions, state[0], s.heads, s.dim,
+                             s.vdim, self.eps, decode=batch.decode_only)
         return ops.linear(y, self.w_o)
 
 

@@ -82,6 +82,16 @@ def rotate_interleaved(x: torch.Tensor, positions: torch.Tensor, freq: torch.Ten
     return torch.stack([u * cos - v * sin, v * cos + u * sin], dim=-1).flatten(-2)
 
 
+def rotate_halves(x: torch.Tensor, positions: torch.Tensor, freq: torch.Tensor) -> torch.Tensor:
+    """CPU restatement of the rotation of pairs (i, i + dims/2): x [T, ..., dims = 2 * len(freq)] fp32."""
+    ang = positions.to(torch.float32).unsqueeze(-1) * freq
+    cos, sin = torch.cos(ang), torch.sin(ang)
+    while cos.dim() < x.dim():
+        cos, sin = cos.unsqueeze(1), sin.unsqueeze(1)
+    u, v = x.chunk(2, dim=-1)
+    return torch.cat([u * cos - v * sin, v * cos + u * sin], dim=-1)
+
+
 def embed_scale(tokens: torch.Tensor, table: torch.Tensor, scale: float) -> Tuple[torch.Tensor, torch.Tensor]:
     """``x = table[tokens] * scale`` -> (fp32 residual stream, the same in the table's type)."""
     T, W = tokens.numel(), table.shape[1]

@@ -62,22 +62,24 @@ def gla_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tensor,
     return out.reshape(T, H * e)
 
 
-def gla_output(o: torch.Tensor, w: torch.Tensor, gate: torch.Tensor, H: int, e: int, eps: float, out_dtype: torch.dtype,
+def gla_output(o: torch.Tensor, w: Optional[torch.Tensor], gate: torch.Tensor, H: int, e: int, eps: float, out_dtype: torch.dtype,
                gate_act: str = "silu") -> torch.Tensor:
-    """``o / sqrt(mean(o^2) + eps) * w * act(gate)`` per (token, head); o: fp32 [T, H e]; w: fp32 [e] (shared by the heads) or
-    [H e]; gate: [T, H e] pre-activation (unit column stride); ``gate_act``: "silu" or "sigmoid".  Returns [T, H e] in
+    """``o / sqrt(mean(o^2) + eps) * w * act(gate)`` per (token, head); o: fp32 [T, H e]; w: fp32 [e] (shared by the heads),
+    [H e] or None (no weight); gate: [T, H e] pre-activation (unit column stride); ``gate_act``: "silu" or "sigmoid".  Returns [T, H e] in
     ``out_dtype``."""
     T = o.shape[0]
-    assert gate_act in ("silu", "sigmoid") and w.numel() in (e, H * e)
-    per_head = w.numel() != e
+    assert gate_act in ("silu", "sigmoid") and (w is None or w.numel() in (e, H * e))
+    per_head = w is not None and w.numel() != e
     if o.is_cuda:
         assert o.is_contiguous() and gate.stride(1) == 1 and gate.dtype == out_dtype
         out = torch.empty(T, H * e, dtype=out_dtype, device=o.device)
-        native.call("llmctl_gla_output", o.data_ptr(), w.data_ptr(), e if per_head else 0, gate.data_ptr(), gate.stride(0),
+        native.call("llmctl_gla_output", o.data_ptr(), native.ptr(w), e if per_head else 0, gate.data_ptr(), gate.stride(0),
                     int(gate_act == "sigmoid"), out.data_ptr(), T, H, e, float(eps), int(out_dtype == torch.float32), native.stream_ptr())
         return out
     oh = o.view(T, H, e)
-    y = oh / torch.sqrt(oh.pow(2).mean(-1, keepdim=True) + eps) * (w.view(H, e) if per_head else w)
+    y = oh / torch.sqrt(oh.pow(2).mean(-1, keepdim=True) + eps)
+    if w is not None:
+        y = y * (w.view(H, e) if per_head else w)
     g = gate.float()
     return (y.reshape(T, H * e) * (F.silu(g) if gate_act == "silu" else torch.sigmoid(g))).to(out_dtype)
 

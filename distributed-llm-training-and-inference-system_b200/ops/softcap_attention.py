@@ -1,11 +1,11 @@
-"""Soft-capped sliding-window attention with kept first tokens, a distance bias and a sink over a paged cache —
+"""Soft-capped sliding-window or chunked attention with kept first tokens, a distance bias and a sink over a paged cache —
 csrc/attention/softcap_window_attention.cu.
 
 ``window_kv_append``: from a packed projection ``[q | k | v | ...]``: fp32 biases, unit-RMS norm of every value head and of
 every query / key head, query temperature, q in fp32, ``[k | v]`` into the token's cache row (``[pages, bs, G d + G e]``).
 ``bucket_bias_table``: a learned bias per logarithmic distance bucket as a table by distance.
-``softcap_window_attention``: for query position i of head h and key position j <= i that is seen (``i - j < window`` or
-``j < keep_first``; ``window`` 0 sees everything):
+``softcap_window_attention``: for query position i of head h and key position j <= i that is seen (``i - j < window`` and in
+the same chunk ``i // chunk == j // chunk``, or ``j < keep_first``; 0: no window / no chunks):
 
     s = q . k * scale;   cap > 0: s <- cap tanh(s / cap);   s <- s - slopes[h] (i - j)
     s <- s + table[h, min(i - j, L - 1)]                                 (no such bias when ``table`` is None)
@@ -35,7 +35,7 @@ native.register_signature("llmctl_window_kv_append", [c_void_p, c_ll, c_void_p, 
 native.register_signature("llmctl_softcap_attention_heads_per_cta", [c_int, c_int, c_int, c_int])
 native.register_signature("llmctl_softcap_attention_mma_ok", [c_int, c_int, c_int, c_int, c_int])
 native.register_signature("llmctl_softcap_window_attention", [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_ll,
-                                                               c_void_p, c_void_p, c_void_p, c_int, c_float, c_float, c_int, c_int, c_int, c_int, c_int, c_int,
+                                                               c_void_p, c_void_p, c_void_p, c_int, c_float, c_float, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                                                                c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p])
 native._KERNELS_PER_CALL["llmctl_softcap_attention_heads_per_cta"] = 0
 native._KERNELS_PER_CALL["llmctl_softcap_attention_mma_ok"] = 0
@@ -137,7 +137,7 @@ def softcap_window_attention(q: torch.Tensor, cache: torch.Tensor, block_tables:
                              positions: torch.Tensor, gate: Optional[torch.Tensor], slopes: Optional[torch.Tensor],
                              sinks: Optional[torch.Tensor], scale: float, cap: float, window: int, keep_first: int, H: int, G: int,
                              d: int, e: int, block_size: int, out_dtype: torch.dtype, max_context: int = 0, splits: int = 0,
-                             tensor_cores: bool = True, table: Optional[torch.Tensor] = None) -> torch.Tensor:
+                             tensor_cores: bool = True, table: Optional[torch.Tensor] = None, chunk: int = 0) -> torch.Tensor:
     """q: fp32 [T, H d]; tiles: int32 [n, 4] = (first token row, tokens <= tile_tokens, block-table row, 0), the tokens of a
     tile being consecutive positions of one sequence; gate: [T, H e] pre-sigmoid (a view with unit column stride) or None;
     slopes, sinks: fp32 [H] or None; table: fp32 [H, L] biases by distance or None.  ``tile_tokens``: 1 (every tile is one decoded token), up to 16, or — where
@@ -158,12 +158,13 @@ def softcap_window_attention(q: torch.Tensor, cache: torch.Tensor, block_tables:
             splits = 1                      # prompt tiles fill the tensor-core kernel's CTAs by themselves
         elif not splits:
             seen = min(max_context, window + keep_first) if window > 0 else max_context
+            seen = min(seen, chunk + keep_first) if chunk > 0 else seen
             splits = key_splits(n * (H // hb), seen, 8 if mma else 2, 64 if mma else 128)
         part_ml = torch.empty(n * (H // hb) * splits * 64, dtype=torch.float32, device=q.device) if splits > 1 else None
         part_o = torch.empty(n * (H // hb) * splits * 32 * e, dtype=torch.float32, device=q.device) if splits > 1 else None
         native.call("llmctl_softcap_window_attention", q.data_ptr(), cache.data_ptr(), block_tables.data_ptr(), block_tables.shape[1],
                     tiles.data_ptr(), n, int(tile_tokens), positions.data_ptr(), native.ptr(gate), gate.stride(0) if gate is not None else 0,
-                    native.ptr(slopes), native.ptr(sinks), native.ptr(table), table.shape[1] if table is not None else 0, float(scale), float(cap), int(window), int(keep_first), H, G, d, e, bs,
+                    native.ptr(slopes), native.ptr(sinks), native.ptr(table), table.shape[1] if table is not None else 0, float(scale), float(cap), int(window), int(keep_first), int(chunk), H, G, d, e, bs,
                     out.data_ptr(), int(splits), native.ptr(part_ml), native.ptr(part_o), _is32(cache), int(mma), native.stream_ptr())
         return out
     out = torch.zeros(T, H, e, dtype=torch.float32)
@@ -174,7 +175,7 @@ def softcap_window_attention(q: torch.Tensor, cache: torch.Tensor, block_tables:
         pages = block_tables[seq]
         for t in range(t0, t0 + n):
             i = int(positions[t])
-            js = [j for j in range(i + 1) if window <= 0 or i - j < window or j < keep_first]
+            js = [j for j in range(i + 1) if j < keep_first or ((window <= 0 or i - j < window) and (chunk <= 0 or i // chunk == j // chunk))]
             kv = flat[[int(pages[j // bs]) * bs + j % bs for j in js]]
             k = kv[:, :G * d].reshape(-1, G, d).repeat_interleave(rep, dim=1)               # [n, H, d]
             v = kv[:, G * d:].reshape(-1, G, e).repeat_interleave(rep, dim=1)               # [n, H, e]

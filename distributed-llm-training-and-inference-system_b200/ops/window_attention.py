@@ -3,8 +3,9 @@
 A query at position i sees the tokens j with ``0 <= i - j < S`` and one pooled key/value (the mean of the cached keys /
 values) per block of P tokens that lies wholly before its window.  A layer's cache is ``[pages, bs + PS, G (d + e)]``:
 ``bs`` token rows ``[keys | values]`` per page, then the ``PS = ceil(bs / P)`` pooled rows of the blocks that start in
-the page.  ``window_qkv_write`` post-processes the packed projection (bias, whole-projection RMS norm of q and k,
-partial interleaved rotation, value mixing with an earlier layer's values) and appends to the cache;
+the page.  ``window_qkv_write`` (csrc/attention/qkv_write.cu) post-processes the packed projection (bias,
+whole-projection RMS norm of q and k, partial rotation of neighbouring pairs or of halves, value mixing with an earlier
+layer's values) and appends to the cache, also for caches without pooled rows;
 ``window_pool_update`` writes the pooled rows of the blocks a step completes; ``pooled_window_attention`` is the
 attention itself, with per-head score temperatures and mixing of the normalised weights across heads.  CPU tensors run
 the PyTorch restatement below (CPU tests); on a GPU a missing kernel raises.
@@ -18,10 +19,10 @@ from typing import Optional
 import torch
 
 from . import native
-from .elementwise import _is32, rotate_interleaved
+from .elementwise import _is32, rotate_halves, rotate_interleaved
 
 c_void_p, c_int, c_ll, c_float = native.c_void_p, native.c_int, native.c_ll, native.c_float
-native.register_signature("llmctl_window_qkv_write", [c_void_p, c_ll, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
+native.register_signature("llmctl_window_qkv_write", [c_void_p, c_ll, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                                                        c_void_p, c_float, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
                                                        c_void_p, c_int, c_void_p, c_int, c_int, c_void_p])
 native.register_signature("llmctl_window_pool_update", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
@@ -55,9 +56,11 @@ def _token_row(table, j: int, bs: int, PS: int) -> int:
 def window_qkv_write(qkv: torch.Tensor, bias: Optional[torch.Tensor], qn_w: Optional[torch.Tensor], kn_w: Optional[torch.Tensor],
                      H: int, G: int, d: int, e: int, rot: int, freq: torch.Tensor, mult: float, eps: float,
                      positions: torch.Tensor, slots: torch.Tensor, cache: torch.Tensor, block_size: int,
-                     v_first: Optional[torch.Tensor] = None, v_mode: int = 0, lam: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """qkv: [T, H d + G d + G e] packed projection WITHOUT bias; bias: same width or None; qn_w / kn_w: fp32 weights of
-    the RMS norm over the whole q / k projection (None = no norm); rot: rotated numbers per head.  ``v_mode`` 1 stores
+                     v_first: Optional[torch.Tensor] = None, v_mode: int = 0, lam: Optional[torch.Tensor] = None,
+                     rot_half: bool = False) -> torch.Tensor:
+    """qkv: [T, >= H d + G d + G e] packed projection WITHOUT bias; bias: fp32 or qkv's type, or None; qn_w / kn_w: fp32
+    weights of the RMS norm over the whole q / k projection (None = no norm); rot: rotated numbers per head, as pairs
+    (2i, 2i + 1) or, with ``rot_half``, (i, i + rot/2).  ``v_mode`` 1 stores
     this layer's values in ``v_first`` [T, G e]; 2 caches ``(1 - lam) v + lam v_first``.  Returns q: fp32 [T, H d];
     writes ``[k | v]`` into ``cache`` ([pages, bs + PS, G (d + e)]) at ``slots`` (int64, page * bs + offset; negative =
     skip)."""
@@ -67,11 +70,11 @@ def window_qkv_write(qkv: torch.Tensor, bias: Optional[torch.Tensor], qn_w: Opti
     if qkv.is_cuda:
         assert qkv.stride(1) == 1 and cache.is_contiguous() and cache.dtype == qkv.dtype
         q = torch.empty(T, Nq, dtype=torch.float32, device=qkv.device)
-        native.call("llmctl_window_qkv_write", qkv.data_ptr(), qkv.stride(0), native.ptr(bias), native.ptr(qn_w), native.ptr(kn_w),
-                    H, G, d, e, rot, native.ptr(freq), float(mult), float(eps), positions.data_ptr(), slots.data_ptr(), q.data_ptr(),
+        native.call("llmctl_window_qkv_write", qkv.data_ptr(), qkv.stride(0), native.ptr(bias), _is32(bias) if bias is not None else 0,
+                    native.ptr(qn_w), native.ptr(kn_w), H, G, d, e, rot, int(rot_half), native.ptr(freq), float(mult), float(eps), positions.data_ptr(), slots.data_ptr(), q.data_ptr(),
                     cache.data_ptr(), bs, PS, native.ptr(v_first), int(v_mode), native.ptr(lam), T, _is32(qkv), native.stream_ptr())
         return q
-    f = qkv.float()
+    f = qkv[:, :Nq + Nk + Nv].float()
     if bias is not None:
         f = f + bias.float()
 
@@ -80,8 +83,9 @@ def window_qkv_write(qkv: torch.Tensor, bias: Optional[torch.Tensor], qn_w: Opti
     q = norm(f[:, :Nq], qn_w).reshape(T, H, d).clone()
     k = norm(f[:, Nq:Nq + Nk], kn_w).reshape(T, G, d).clone()
     if rot:
-        q[..., :rot] = rotate_interleaved(q[..., :rot], positions, freq, mult)
-        k[..., :rot] = rotate_interleaved(k[..., :rot], positions, freq, mult)
+        def turn(x):
+            return rotate_halves(x, positions, freq) * mult if rot_half else rotate_interleaved(x, positions, freq, mult)
+        q[..., :rot], k[..., :rot] = turn(q[..., :rot]), turn(k[..., :rot])
     v = f[:, Nq + Nk:].to(qkv.dtype)
     if v_mode == 1:
         v_first.copy_(v)

@@ -134,8 +134,9 @@ class RaggedBatch:
         up to ``rows`` heads when every sequence decodes."""
         return min(heads, rows) if self.decode_only else 1
 
-    def attention_splits(self, heads: int, rows: int = ROWS_PER_TILE) -> int:
-        """Split the keys of long contexts over CTAs when the tiles alone would leave most SMs idle."""
+    def attention_splits(self, heads: int, rows: int = ROWS_PER_TILE, span: Optional[int] = None) -> int:
+        """Split the keys of long contexts over CTAs when the tiles alone would leave most SMs idle.  ``span``: most keys a
+        tile reads (the longest context unless a window bounds it)."""
         hpt = self.heads_per_tile(heads, rows)
         ctas = self._tiles[rows].shape[0] * ((heads + hpt - 1) // hpt)
-        return int(max(1, min(2 * self._sms // max(ctas, 1), self.max_context // 64)))
+        return int(max(1, min(2 * self._sms // max(ctas, 1), (self.max_context if span is None else span) // 64)))

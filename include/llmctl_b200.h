@@ -235,23 +235,27 @@ int llmctl_latent_attention(const void* ql, int ql_bf16, long long ql_st, long l
                             const int* tiles, int ntiles, int tokens, const int* positions, const float* freq, float mult,
                             float scale, int H, int R, int dr, int heads_per_tile, int splits, int keys_per_split,
                             void* out, float* partial, int is_fp32, int tensor_cores, int rows_per_tile,
-                            const float* sinks /* fp32 [H] or null: exp(sinks[h]) joins head h's softmax denominator */, void* stream);
+                            const float* sinks /* fp32 [H] or null: exp(sinks[h]) joins head h's softmax denominator */,
+                            int window /* 0: every earlier key */, const void* head_gate /* [tokens, H] pre-sigmoid or null */,
+                            long long gate_ld, void* stream);
 /* The tcgen05 kernel (128-row query tiles): sizes that qualify, status of its bounded waits, and the launch.
- * qfull: bf16 scratch [tokens, H, R + dr]; cache_rows = blocks x block_size. */
+ * qfull: bf16 scratch [tokens, H, R + dr], or null when dr is 0 and ql is bf16 [heads, tokens, R]; cache_rows = blocks x block_size. */
 int llmctl_latent_attention_t5_ok(int R, int dr, int block_size);
 int llmctl_latent_attention_t5_status(int clear);
 int llmctl_latent_attention_t5(const void* ql, int ql_bf16, long long ql_st, long long ql_sh, const void* q, long long ldq,
                                int dn, const void* cache, long long cache_rows, const int* block_tables, int max_blocks,
                                int block_size, const int* tiles, int ntiles, int tokens, const int* positions,
                                const float* freq, float mult, float scale, int H, int R, int dr, int heads_per_tile,
-                               int splits, int keys_per_split, void* qfull, void* out, float* partial, const float* sinks, void* stream);
+                               int splits, int keys_per_split, void* qfull, void* out, float* partial, const float* sinks, int window,
+                               const void* head_gate, long long gate_ld, void* stream);
 int llmctl_moe_tile_rows(void);
 /* correction: fp32 [E] added to the scores for the CHOICE only, or null; n_groups > 1: only experts of the keep_groups
- * best groups (of E / n_groups neighbours each) can be chosen.  Ids >= the E given to plan / permute are identity
+ * best groups (of E / n_groups neighbours each) can be chosen, a group's score being its best (group_best 1) or the sum of
+ * its two best (2) choice scores; weights are multiplied by weight_scale.  Ids >= the E given to plan / permute are identity
  * experts. */
 int llmctl_moe_route(const float* x, const void* wr, const void* wg, int is_fp32, int tokens, int W, int E, int top,
-                     int softmax_scores, int renormalise, const float* correction, int n_groups, int keep_groups, int* ids,
-                     float* weights, float* gate, int* counts, void* stream);
+                     int softmax_scores, int renormalise, const float* correction, int n_groups, int keep_groups, int group_best,
+                     float weight_scale, int* ids, float* weights, float* gate, int* counts, void* stream);
 /* meta: int32 [2 E + 2 + max_tiles] = { segment offsets[E] | cursors[E] | tiles | padded rows | tile -> expert }. */
 int llmctl_moe_plan(const int* counts, int E, int* meta, int max_tiles, int tile_rows, void* stream);
 int llmctl_moe_permute(const float* x, int W, const int* ids, const float* weights, int scale_input, int* meta, int E,
@@ -281,9 +285,9 @@ int llmctl_rmsnorm_rows(const float* x, const long long* rows, const float* w, v
 int llmctl_sandwich_residual(const void* y, int y_fp32, long long ldy, float* x, const float* wb, const float* w_next,
                              void* out, int out_fp32, float* out32, int rows, int cols, float eps, void* stream);
 /* Packed projection [q | k | v] -> fp32 queries and the token's cache row: bias, RMS norm over the whole q / k
- * projection, rotation of the first `rot` numbers of every head, value mixing (v_mode 1: publish v_first, 2: blend). */
-int llmctl_window_qkv_write(const void* qkv, long long ld, const void* bias, const float* qn_w, const float* kn_w, int H,
-                            int G, int d, int e, int rot, const float* freq, float mult, float eps, const int* positions,
+ * projection, rotation of the first `rot` numbers of every head (neighbouring pairs, or (i, i + rot/2) if rot_half), value mixing (v_mode 1: publish v_first, 2: blend). */
+int llmctl_window_qkv_write(const void* qkv, long long ld, const void* bias, int bias_fp32, const float* qn_w, const float* kn_w, int H,
+                            int G, int d, int e, int rot, int rot_half, const float* freq, float mult, float eps, const int* positions,
                             const long long* slots, float* q_out, void* cache, int bs, int PS, void* v_first, int v_mode,
                             const float* lam, int tokens, int is_fp32, void* stream);
 /* Pooled rows (means of P cached rows) of the blocks that the step's tokens complete. */
@@ -364,12 +368,12 @@ int llmctl_window_kv_append(const void* proj, long long ld, const float* bias, i
                             const long long* slots, float* q_out, void* cache, int tokens, int is_fp32, void* stream);
 int llmctl_softcap_attention_heads_per_cta(int H, int G, int tile_tokens, int use_mma);
 int llmctl_softcap_attention_mma_ok(int H, int G, int d, int e, int tile_tokens);
-/* Sliding window (0: none) with kept first tokens, tanh soft cap (0: none), per-head distance slopes and sinks (null:
+/* Sliding window (0: none) with kept first tokens, chunks counted from position 0 (0: none), tanh soft cap (0: none), per-head distance slopes and sinks (null:
  * none), table of biases by distance [H, table_len] (null: none), sigmoid output gate (null: none). */
 int llmctl_softcap_window_attention(const float* q, const void* cache, const int* block_tables, int max_blocks, const int* tiles,
                                     int ntiles, int tile_tokens, const int* positions, const void* gate, long long gate_ld,
                                     const float* slopes, const float* sinks, const float* table, int table_len, float scale,
-                                    float cap, int window, int keep_first, int H, int G, int d, int e, int bs, void* out,
+                                    float cap, int window, int keep_first, int chunk, int H, int G, int d, int e, int bs, void* out,
                                     int splits, float* part_ml, float* part_o, int is_fp32, int use_mma, void* stream);
 
 /* ---- two-norm parallel layers, matrix-state recurrences (csrc/norm/dual_norm.cu, csrc/recurrent/matrix_state.cu) ---- */
@@ -399,6 +403,26 @@ int llmctl_matrix_step(const void* x, long long ldx, const void* r, long long ld
 int llmctl_token_shift(const void* h, const float* mu, int n_mix, const int* portions, const int* seq_rows, float* state, void* out,
                        int tokens, int W, int is_fp32, void* stream);
 int llmctl_tanh(void* z, long long ld, int is_fp32, int rows, int F, void* stream);
+
+/* ---- hyper-connected streams, retention (csrc/norm/hyper_norm.cu, csrc/recurrent/retention.cu) ---- */
+/* x_t <- sum_s mix[s, t] x_s + out_w[t] y on the fp32 streams [T, S, W] (y null: unchanged), and the layer norm of
+ * sum_t in_w[t] x_t (in_w null: ones; w null: none); rows: only the norms of those tokens, nothing written back. */
+int llmctl_hyper_step(float* x, int S, const void* y, int y_fp32, long long ldy, const float* mix, const float* out_w,
+                      const float* in_w, const float* w, const float* b, void* out, int out_fp32, float* out32,
+                      const long long* rows, int n, int W, float eps, void* stream);
+/* x_s[t] = scale * table[tokens[t]] for every stream s, and the first norm. */
+int llmctl_hyper_embed(const long long* tokens, const void* table, int is_fp32, float scale, float* x, int S, const float* in_w,
+                       const float* w, const float* b, void* out, float* out32, int T, int W, float eps, void* stream);
+/* Retention: rotation by halves, S <- decay S + k v^T, o = S^T q (scan over a prepare pass); the single-launch step. */
+int llmctl_retention_prepare(const void* q, long long ldq, const void* k, long long ldk, const void* v, long long ldv,
+                             const int* positions, const float* freq, int rot, const float* decay_m1, int tokens, float* work,
+                             int H, int d, int e, int is_fp32, void* stream);
+int llmctl_retention_scan(float* work, const int* portions, int nportions, int tokens, float* state, float* out, int H, int d, int e,
+                          void* stream);
+int llmctl_retention_step(const void* q, long long ldq, const void* k, long long ldk, const void* v, long long ldv,
+                          const int* positions, const float* freq, int rot, const float* decay_m1, const int* portions,
+                          int nportions, float* state, const void* gate, long long ldg, int gate_kind, float eps, void* out, int H,
+                          int d, int e, int is_fp32, void* stream);
 
 #ifdef __cplusplus
 }
