@@ -26,30 +26,54 @@ xielu_kernel(const T* __restrict__ z, T* __restrict__ out, long long n, float a_
   }
 }
 
+// x * sigmoid(z).  bf16 operands carry 8 bits, so the hardware's exponential and reciprocal are exact enough there.
 template <typename T>
-__global__ void __launch_bounds__(256)
-gated_silu_kernel(const T* __restrict__ gu, long long ld, T* __restrict__ out, int rows, int F) {
-  const long long n = static_cast<long long>(rows) * F;
-  for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < n;
-       i += static_cast<long long>(gridDim.x) * blockDim.x) {
-    const long long r = i / F;
-    const int c = static_cast<int>(i % F);
-    const float g = to_f32(gu[r * ld + c]), u = to_f32(gu[r * ld + F + c]);
-    out[i] = from_f32<T>(g / (1.f + expf(-g)) * u);
-  }
+__device__ __forceinline__ float times_sigmoid(float x, float z) {
+  if (sizeof(T) == 2) return __fdividef(x, 1.f + __expf(-fmaxf(z, -80.f)));
+  return x / (1.f + expf(-z));
 }
 
-// tanh form of GELU on the gate of a packed [gate | up] activation: 0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3))) * up
 template <typename T>
+struct GateSilu {
+  __device__ __forceinline__ float operator()(float g, float u) const { return times_sigmoid<T>(g, g) * u; }
+};
+// tanh form of GELU: 0.5 g (1 + tanh(y)) = g sigmoid(2 y), y = sqrt(2/pi) (g + 0.044715 g^3)
+template <typename T>
+struct GateGelu {
+  __device__ __forceinline__ float operator()(float g, float u) const {
+    return times_sigmoid<T>(g, 1.5957691216057308f * (g + 0.044715f * g * g * g)) * u;
+  }
+};
+template <typename T>
+struct GateClamped {
+  float limit, alpha;
+  __device__ __forceinline__ float operator()(float g, float u) const {
+    g = fminf(g, limit);
+    return times_sigmoid<T>(g, alpha * g) * (fminf(fmaxf(u, -limit), limit) + 1.f);
+  }
+};
+
+// out = act(gate, up) on a packed [rows, 2F] activation (gate first, row stride ld).  VEC: numbers per step (8: 16 or 32 bytes).
+template <typename T, int VEC, typename Act>
 __global__ void __launch_bounds__(256)
-gated_gelu_tanh_kernel(const T* __restrict__ gu, long long ld, T* __restrict__ out, int rows, int F) {
-  const long long n = static_cast<long long>(rows) * F;
-  for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < n;
+gated_kernel(const T* __restrict__ gu, long long ld, T* __restrict__ out, long long groups, int F, Act act) {
+  const int per_row = F / VEC;
+  for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < groups;
        i += static_cast<long long>(gridDim.x) * blockDim.x) {
-    const long long r = i / F;
-    const int c = static_cast<int>(i % F);
-    const float g = to_f32(gu[r * ld + c]), u = to_f32(gu[r * ld + F + c]);
-    out[i] = from_f32<T>(0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u);
+    const long long r = groups <= 0x7fffffffLL ? static_cast<unsigned>(i) / static_cast<unsigned>(per_row) : i / per_row;
+    const int c = static_cast<int>(i - r * per_row) * VEC;
+    const T* g = gu + r * ld + c;
+    T* o = out + r * F + c;
+    if constexpr (VEC == 1) {
+      o[0] = from_f32<T>(act(to_f32(g[0]), to_f32(g[F])));
+    } else {
+      float a[VEC], b[VEC];
+      load8_f32(g, a);
+      load8_f32(g + F, b);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) a[j] = act(a[j], b[j]);
+      store8_f32(o, a);
+    }
   }
 }
 
@@ -63,20 +87,6 @@ sigmoid_gate_kernel(T* __restrict__ y, const T* __restrict__ z, long long ldz, i
     const long long r = i / F;
     const int c = static_cast<int>(i % F);
     y[i] = from_f32<T>(to_f32(y[i]) / (1.f + expf(-to_f32(z[r * ldz + c]))));
-  }
-}
-
-template <typename T>
-__global__ void __launch_bounds__(256)
-gated_clamped_kernel(const T* __restrict__ gu, long long ld, T* __restrict__ out, int rows, int F, float limit, float alpha) {
-  const long long n = static_cast<long long>(rows) * F;
-  for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < n;
-       i += static_cast<long long>(gridDim.x) * blockDim.x) {
-    const long long r = i / F;
-    const int c = static_cast<int>(i % F);
-    const float g = fminf(to_f32(gu[r * ld + c]), limit);
-    const float u = fminf(fmaxf(to_f32(gu[r * ld + F + c]), -limit), limit);
-    out[i] = from_f32<T>(g / (1.f + expf(-alpha * g)) * (u + 1.f));
   }
 }
 
@@ -106,6 +116,14 @@ static inline int grid_for(long long n) {
   return static_cast<int>(b);
 }
 
+template <typename T, typename Act>
+static void launch_gated(const T* gu, long long ld, T* out, int rows, int F, Act act, cudaStream_t s) {
+  const bool vec = F % 8 == 0 && ld % 8 == 0 && ((reinterpret_cast<uintptr_t>(gu) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+  const long long groups = static_cast<long long>(rows) * F / (vec ? 8 : 1);
+  if (vec) gated_kernel<T, 8, Act><<<grid_for(groups), 256, 0, s>>>(gu, ld, out, groups, F, act);
+  else gated_kernel<T, 1, Act><<<grid_for(groups), 256, 0, s>>>(gu, ld, out, groups, F, act);
+}
+
 }  // namespace llmctl
 
 using namespace llmctl;
@@ -121,8 +139,7 @@ LLMCTL_API int llmctl_gated_silu(const void* gate_up, long long ld, void* out, i
   LLMCTL_BEGIN();
   LLMCTL_REQUIRE(ld >= 2LL * F);
   if (rows == 0 || F == 0) return 0;
-  LLMCTL_DISPATCH_DTYPE(is_fp32, T, (gated_silu_kernel<T><<<grid_for(static_cast<long long>(rows) * F), 256, 0, (cudaStream_t)stream>>>(
-                                        (const T*)gate_up, ld, (T*)out, rows, F)));
+  LLMCTL_DISPATCH_DTYPE(is_fp32, T, (launch_gated<T>((const T*)gate_up, ld, (T*)out, rows, F, GateSilu<T>{}, (cudaStream_t)stream)));
   LLMCTL_RETURN_LAST();
 }
 
@@ -130,8 +147,7 @@ LLMCTL_API int llmctl_gated_gelu_tanh(const void* gate_up, long long ld, void* o
   LLMCTL_BEGIN();
   LLMCTL_REQUIRE(ld >= 2LL * F);
   if (rows == 0 || F == 0) return 0;
-  LLMCTL_DISPATCH_DTYPE(is_fp32, T, (gated_gelu_tanh_kernel<T><<<grid_for(static_cast<long long>(rows) * F), 256, 0, (cudaStream_t)stream>>>(
-                                        (const T*)gate_up, ld, (T*)out, rows, F)));
+  LLMCTL_DISPATCH_DTYPE(is_fp32, T, (launch_gated<T>((const T*)gate_up, ld, (T*)out, rows, F, GateGelu<T>{}, (cudaStream_t)stream)));
   LLMCTL_RETURN_LAST();
 }
 
@@ -149,8 +165,7 @@ LLMCTL_API int llmctl_gated_clamped(const void* gate_up, long long ld, void* out
   LLMCTL_BEGIN();
   LLMCTL_REQUIRE(ld >= 2LL * F && limit > 0.f);
   if (rows == 0 || F == 0) return 0;
-  LLMCTL_DISPATCH_DTYPE(is_fp32, T, (gated_clamped_kernel<T><<<grid_for(static_cast<long long>(rows) * F), 256, 0, (cudaStream_t)stream>>>(
-                                        (const T*)gate_up, ld, (T*)out, rows, F, limit, alpha)));
+  LLMCTL_DISPATCH_DTYPE(is_fp32, T, (launch_gated<T>((const T*)gate_up, ld, (T*)out, rows, F, GateClamped<T>{limit, alpha}, (cudaStream_t)stream)));
   LLMCTL_RETURN_LAST();
 }
 

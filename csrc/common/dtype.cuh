@@ -46,6 +46,18 @@ __device__ __forceinline__ void store_vec(__nv_bfloat16* p, const float (&v)[VEC
   else p[0] = __float2bfloat16(v[0]);
 }
 
+// Eight neighbouring numbers (16-byte aligned addresses).
+__device__ __forceinline__ void load8_f32(const __nv_bfloat16* p, float (&v)[8]) { unpack8(load8(p), v); }
+__device__ __forceinline__ void load8_f32(const float* p, float (&v)[8]) {
+  *reinterpret_cast<float4*>(v) = *reinterpret_cast<const float4*>(p);
+  *reinterpret_cast<float4*>(v + 4) = *reinterpret_cast<const float4*>(p + 4);
+}
+__device__ __forceinline__ void store8_f32(__nv_bfloat16* p, const float (&v)[8]) { store8(p, pack8(v)); }
+__device__ __forceinline__ void store8_f32(float* p, const float (&v)[8]) {
+  *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  *reinterpret_cast<float4*>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
+}
+
 }  // namespace llmctl
 
 // Dispatch a templated launch on the `is_fp32` flag of the C ABI.

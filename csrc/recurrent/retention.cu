@@ -9,6 +9,14 @@
 //   llmctl_retention_scan : the serial part (the matrix-state scan, kind 3; any sizes).
 //   llmctl_retention_step : one decoded token per sequence in ONE launch: rotation, state update, read-out, the head's RMS norm
 //       and output gate.
+//   llmctl_retention_chunked : prompts in bf16 (sizes below), chunks of 64 tokens as matrix products on the tensor cores
+//       (mma.sync m16n8k16) instead of the serial scan.  With local indices i, j in a chunk of L tokens and S before it:
+//           o_i = decay^(i+1) q_i^T S + sum_(j <= i) decay^(i-j) (q_i . k_j) v_j
+//           S  <- decay^L S + sum_j decay^(L-1-j) k_j v_j^T
+//       Four launches: sines and cosines per (token, pair); the sums over j of every chunk and head (parallel); the chain over the
+//       chunks, elementwise in fp32, which leaves the state before every chunk; outputs with the head's RMS norm and gate
+//       (parallel).  Rotated queries and keys, decayed scores and states enter the products as bf16 pairs hi + lo (exact to
+//       ~2^-17; values are bf16 already), accumulators and the carried state are fp32.
 // The decay is applied as S + (decay - 1) S.  Everything is fp32; only the projections and the gated output have the activation type.
 // Reference: none (the reference has no model code).
 #include "matrix_state.cuh"
@@ -77,6 +85,370 @@ retention_prepare_kernel(const RetentionPrepParams p) {
   }
 }
 
+// ---------------------------------------------------------------------------------------------------------------
+// chunks of 64 tokens on the tensor cores
+// ---------------------------------------------------------------------------------------------------------------
+constexpr int kRcTokens = 64;
+
+struct RetentionChunkParams {
+  const __nv_bfloat16* q;     // [T, H d] (row strides below)
+  const __nv_bfloat16* k;
+  const __nv_bfloat16* v;     // [T, H e]
+  const __nv_bfloat16* gate;  // [T, H e]
+  long long ldq, ldk, ldv, ldg;
+  const float2* cs;           // [T, half] (cos, sin)
+  int half;                   // rotated pairs per head
+  const float* dm;            // [H] decay minus one
+  const int* portions;
+  int nportions;
+  const int* tiles;           // [chunks, 4] = (first token row, tokens, portion, 0), portions in order
+  float* state;               // [slots, H, d, e]
+  float* scratch;             // [chunks, nh, d, e]: a chunk's sum, then groups of 4 numbers of the state before it as 4 hi, 4 lo
+  __nv_bfloat16* out;         // [T, H e]
+  int H, d, e, h0, nh;        // heads h0 .. h0 + nh - 1
+  int gate_sigmoid;
+  float eps;
+};
+
+__global__ void __launch_bounds__(256)
+retention_angles_kernel(const int* __restrict__ positions, const float* __restrict__ freq, int half, float2* __restrict__ cs, int tokens) {
+  const int i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= tokens * half) return;
+  float s, c;
+  sincosf(static_cast<float>(positions[i / half]) * freq[i % half], &s, &c);
+  cs[i] = make_float2(c, s);
+}
+
+__device__ __forceinline__ float rc_log2_decay(float dm) { return log1pf(dm) * 1.4426950408889634f; }
+__device__ __forceinline__ float rc_power(float log2_decay, int n) { return n == 0 ? 1.f : exp2f(log2_decay * static_cast<float>(n)); }
+
+// four fp32 numbers as bf16 pairs hi + lo
+__device__ __forceinline__ void rc_split4(const float (&v)[4], uint2& hi, uint2& lo) {
+  float r[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) r[i] = v[i] - __bfloat162float(__float2bfloat16(v[i]));
+  hi = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]));
+  lo = make_uint2(pack_bf16x2(r[0], r[1]), pack_bf16x2(r[2], r[3]));
+}
+
+// Rows j of a chunk (x + j ld, d numbers): rotated, times factor * decay^(last - j) (log2_decay 0: no decay), split into hi and lo
+// [64][d + 8] in shared memory; rows past n are zeros.
+__device__ __forceinline__ void rc_load_rotated(const __nv_bfloat16* x, long long ld, const float2* cs, int half, int d, int n, float factor,
+                                                float log2_decay, int last, __nv_bfloat16* hi, __nv_bfloat16* lo) {
+  const int per = d >> 2, lds = d + 8;
+  for (int i = threadIdx.x; i < kRcTokens * per; i += blockDim.x) {
+    const int j = i / per, c = (i - j * per) << 2;
+    if (c >= half && c < 2 * half) continue;           // the second number of a pair goes with the first
+    float a[4] = {0.f, 0.f, 0.f, 0.f}, b[4] = {0.f, 0.f, 0.f, 0.f};
+    if (j < n) {
+      const float f = factor * rc_power(log2_decay, last - j);
+      load_vec<4>(x + j * ld + c, a);
+      if (c < half) {
+        load_vec<4>(x + j * ld + c + half, b);
+        float w[8];
+        const float* t = reinterpret_cast<const float*>(cs + static_cast<long long>(j) * half + c);
+        *reinterpret_cast<float4*>(w) = *reinterpret_cast<const float4*>(t);
+        *reinterpret_cast<float4*>(w + 4) = *reinterpret_cast<const float4*>(t + 4);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          const float u = a[k], v = b[k];
+          a[k] = (u * w[2 * k] - v * w[2 * k + 1]) * f;
+          b[k] = (v * w[2 * k] + u * w[2 * k + 1]) * f;
+        }
+      } else {
+#pragma unroll
+        for (int k = 0; k < 4; ++k) a[k] *= f;
+      }
+    }
+    uint2 h, l;
+    rc_split4(a, h, l);
+    *reinterpret_cast<uint2*>(hi + j * lds + c) = h;
+    *reinterpret_cast<uint2*>(lo + j * lds + c) = l;
+    if (c < half) {
+      rc_split4(b, h, l);
+      *reinterpret_cast<uint2*>(hi + j * lds + c + half) = h;
+      *reinterpret_cast<uint2*>(lo + j * lds + c + half) = l;
+    }
+  }
+}
+
+__device__ __forceinline__ void rc_load_rows(const __nv_bfloat16* x, long long ld, int cols, int n, __nv_bfloat16* dst, int lds) {
+  const int per = cols >> 3;
+  for (int i = threadIdx.x; i < kRcTokens * per; i += blockDim.x) {
+    const int j = i / per, c = (i - j * per) << 3;
+    const uint4 u = j < n ? *reinterpret_cast<const uint4*>(x + j * ld + c) : make_uint4(0u, 0u, 0u, 0u);
+    *reinterpret_cast<uint4*>(dst + j * lds + c) = u;
+  }
+}
+
+// A fragment of A[m][k] = s[k0 + k][m0 + m] (operand stored [k][m] row-major): ldmatrix with transposition
+__device__ __forceinline__ void rc_a_frag_km(uint32_t (&a)[4], const __nv_bfloat16* s, int ld, int m0, int k0, int lane) {
+  const __nv_bfloat16* p = s + (k0 + (lane & 7) + ((lane >> 4) << 3)) * ld + m0 + (((lane >> 3) & 1) << 3);
+  const uint32_t addr = static_cast<uint32_t>(__cvta_generic_to_shared(p));
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];\n"
+               : "=r"(a[0]), "=r"(a[1]), "=r"(a[2]), "=r"(a[3])
+               : "r"(addr));
+}
+
+// scratch[chunk, head] = sum_j decay^(L-1-j) k_j v_j^T.  Grid: (chunks, heads); a warp owns blocks of 16 x 32 numbers.
+__global__ void __launch_bounds__(256)
+retention_chunk_sum_kernel(const RetentionChunkParams p) {
+  extern __shared__ __align__(16) unsigned char rc_smem[];
+  const int d = p.d, e = p.e, ldk = d + 8, ldv = e + 8, h = p.h0 + blockIdx.y;
+  const int* tile = p.tiles + 4 * blockIdx.x;
+  const long long t0 = tile[0];
+  const int n = tile[1];
+  if (n <= 0) return;
+  __nv_bfloat16* Kh = reinterpret_cast<__nv_bfloat16*>(rc_smem);
+  __nv_bfloat16* Kl = Kh + kRcTokens * ldk;
+  __nv_bfloat16* V = Kl + kRcTokens * ldk;
+  const float lg = rc_log2_decay(p.dm[h]);
+  rc_load_rotated(p.k + t0 * p.ldk + h * d, p.ldk, p.cs + t0 * p.half, p.half, d, n, 1.f / sqrtf(static_cast<float>(d)), lg, n - 1, Kh, Kl);
+  rc_load_rows(p.v + t0 * p.ldv + h * e, p.ldv, e, n, V, ldv);
+  __syncthreads();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3;
+  const int nb = (e + 31) / 32, blocks = (d / 16) * nb, steps = (n + 15) / 16;
+  float* dst = p.scratch + (static_cast<long long>(blockIdx.x) * p.nh + blockIdx.y) * d * e;
+  for (int b = warp; b < blocks; b += 8) {
+    const int m0 = b / nb * 16, n0 = b % nb * 32;
+    float acc[4][4] = {};
+    for (int ks = 0; ks < steps; ++ks) {
+      uint32_t ah[4], al[4];
+      rc_a_frag_km(ah, Kh, ldk, m0, ks * 16, lane);
+      rc_a_frag_km(al, Kl, ldk, m0, ks * 16, lane);
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        if (n0 + 8 * i < e) {
+          uint32_t bf[2];
+          load_b_frag_kn(bf, V, ldv, ks * 16, n0 + 8 * i, lane);
+          mma_bf16_16816(acc[i], ah, bf);
+          mma_bf16_16816(acc[i], al, bf);
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+      if (n0 + 8 * i < e) {
+        float* o = dst + static_cast<long long>(m0 + g) * e + n0 + 8 * i + 2 * t;
+        *reinterpret_cast<float2*>(o) = make_float2(acc[i][0], acc[i][1]);
+        *reinterpret_cast<float2*>(o + 8 * e) = make_float2(acc[i][2], acc[i][3]);
+      }
+  }
+}
+
+// The chain over a portion's chunks, four numbers of a head's state per thread.  Grid: (portions, heads, d e / 1024).
+__global__ void __launch_bounds__(256)
+retention_chunk_chain_kernel(const RetentionChunkParams p) {
+  constexpr int AHEAD = 4;
+  const int* pt = p.portions + 4 * blockIdx.x;
+  const int n = pt[1], slot = pt[3], h = p.h0 + blockIdx.y;
+  const long long numbers = static_cast<long long>(p.d) * p.e, i = (static_cast<long long>(blockIdx.z) * blockDim.x + threadIdx.x) * 4;
+  if (n <= 0 || i >= numbers) return;
+  int first = 0;
+  for (int b = 0; b < static_cast<int>(blockIdx.x); ++b) first += (max(p.portions[4 * b + 1], 0) + kRcTokens - 1) / kRcTokens;
+  const int chunks = (n + kRcTokens - 1) / kRcTokens;
+  float* st = slot >= 0 ? p.state + (static_cast<long long>(slot) * p.H + h) * numbers + i : nullptr;
+  float4 S = (st && pt[2] > 0) ? *reinterpret_cast<const float4*>(st) : make_float4(0.f, 0.f, 0.f, 0.f);
+  const float lg = log1pf(p.dm[h]);
+  const float full = expm1f(lg * kRcTokens), rest = expm1f(lg * static_cast<float>(n - (chunks - 1) * kRcTokens));
+  const long long step = static_cast<long long>(p.nh) * numbers;
+  float* x = p.scratch + (static_cast<long long>(first) * p.nh + blockIdx.y) * numbers + i;
+  float4 kv[AHEAD];
+#pragma unroll
+  for (int a = 0; a < AHEAD; ++a)
+    if (a < chunks) kv[a] = *reinterpret_cast<const float4*>(x + a * step);
+  for (int c0 = 0; c0 < chunks; c0 += AHEAD) {
+#pragma unroll
+    for (int a = 0; a < AHEAD; ++a) {
+      const int c = c0 + a;
+      if (c >= chunks) break;
+      const float s[4] = {S.x, S.y, S.z, S.w};
+      uint2 hi, lo;
+      rc_split4(s, hi, lo);
+      const float gm = c + 1 < chunks ? full : rest;
+      S.x = fmaf(gm, S.x, S.x) + kv[a].x;
+      S.y = fmaf(gm, S.y, S.y) + kv[a].y;
+      S.z = fmaf(gm, S.z, S.z) + kv[a].z;
+      S.w = fmaf(gm, S.w, S.w) + kv[a].w;
+      *reinterpret_cast<uint4*>(x + c * step) = make_uint4(hi.x, hi.y, lo.x, lo.y);
+      if (c + AHEAD < chunks) kv[a] = *reinterpret_cast<const float4*>(x + (c + AHEAD) * step);
+    }
+  }
+  if (st) *reinterpret_cast<float4*>(st) = S;
+}
+
+// Outputs of a chunk and head.  Warp (r, c) = (warp % 4, warp / 4) owns 16 tokens and half of the value columns (NT tiles of 8).
+template <int NT>
+__global__ void __launch_bounds__(256, NT <= 8 ? 2 : 1)
+retention_chunk_output_kernel(const RetentionChunkParams p) {
+  extern __shared__ __align__(16) unsigned char rc_smem[];
+  __shared__ float row_ss[2][kRcTokens];
+  const int d = p.d, e = p.e, ldq = d + 8, ldv = e + 8, h = p.h0 + blockIdx.y;
+  const int* tile = p.tiles + 4 * blockIdx.x;
+  const long long t0 = tile[0];
+  const int n = tile[1];
+  if (n <= 0) return;
+  const int* pt = p.portions + 4 * tile[2];
+  const bool has_state = t0 > pt[0] || (pt[2] > 0 && pt[3] >= 0);      // the first chunk of a sequence starts from zeros
+  __nv_bfloat16* Qh = reinterpret_cast<__nv_bfloat16*>(rc_smem);
+  __nv_bfloat16* Ql = Qh + kRcTokens * ldq;
+  __nv_bfloat16* V = Ql + kRcTokens * ldq;
+  __nv_bfloat16* Kh = V + kRcTokens * ldv;             // keys, then 64 rows of the state at a time
+  __nv_bfloat16* Kl = Kh + kRcTokens * ldq;
+  __nv_bfloat16* Sh = Kh;
+  __nv_bfloat16* Sl = Sh + kRcTokens * ldv;
+  const float2* cs = p.cs + t0 * p.half;
+  rc_load_rotated(p.q + t0 * p.ldq + h * d, p.ldq, cs, p.half, d, n, 1.f, 0.f, 0, Qh, Ql);
+  rc_load_rotated(p.k + t0 * p.ldk + h * d, p.ldk, cs, p.half, d, n, 1.f / sqrtf(static_cast<float>(d)), 0.f, 0, Kh, Kl);
+  rc_load_rows(p.v + t0 * p.ldv + h * e, p.ldv, e, n, V, ldv);
+  __syncthreads();
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
+  const int rg = warp & 3, r0 = rg * 16, n_base = (warp >> 2) * NT * 8;
+  const bool active = r0 < n;
+  const float lg = rc_log2_decay(p.dm[h]);
+  uint32_t ph[4][4], pl[4][4];                         // decayed scores, A fragments of 16 keys each
+  if (active) {
+    float s[8][4];
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) s[i][j] = 0.f;
+    for (int ks = 0; ks < d; ks += 16) {
+      uint32_t ah[4], al[4];
+      load_a_frag(ah, Qh, ldq, r0, ks, lane);
+      load_a_frag(al, Ql, ldq, r0, ks, lane);
+#pragma unroll
+      for (int i = 0; i < 8; ++i)
+        if (i < 2 * (rg + 1)) {                        // later keys are masked for all rows of the warp
+          uint32_t bh[2], bl[2];
+          load_b_frag_nk(bh, Kh, ldq, 8 * i, ks, lane);
+          load_b_frag_nk(bl, Kl, ldq, 8 * i, ks, lane);
+          mma_bf16_16816(s[i], ah, bh);
+          mma_bf16_16816(s[i], al, bh);
+          mma_bf16_16816(s[i], ah, bl);
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int dist = r0 + g + (j >> 1) * 8 - (8 * i + 2 * t + (j & 1));
+        s[i][j] = dist >= 0 ? s[i][j] * rc_power(lg, dist) : 0.f;
+      }
+#pragma unroll
+    for (int kk = 0; kk < 4; ++kk)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {                    // fragment register j: rows g (+8 for odd j), keys 2t, 2t + 1 (+8 for j >= 2)
+        const float a = s[2 * kk + (j >> 1)][(j & 1) * 2], b = s[2 * kk + (j >> 1)][(j & 1) * 2 + 1];
+        const float ra = a - __bfloat162float(__float2bfloat16(a)), rb = b - __bfloat162float(__float2bfloat16(b));
+        ph[kk][j] = pack_bf16x2(a, b);
+        pl[kk][j] = pack_bf16x2(ra, rb);
+      }
+  }
+  float acc[NT][4];
+#pragma unroll
+  for (int i = 0; i < NT; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+  if (has_state) {                                     // uniform over the CTA
+    const uint4* src = reinterpret_cast<const uint4*>(p.scratch + (static_cast<long long>(blockIdx.x) * p.nh + blockIdx.y) * d * e);
+    const int per = e >> 2;
+    for (int ds = 0; ds < d; ds += kRcTokens) {
+      const int rows = min(kRcTokens, d - ds);
+      __syncthreads();                                 // the readers of the keys / the previous rows are done
+      for (int i = tid; i < rows * per; i += 256) {
+        const int r = i / per, c = (i - r * per) << 2;
+        const uint4 u = src[static_cast<long long>(ds + r) * per + (c >> 2)];
+        *reinterpret_cast<uint2*>(Sh + r * ldv + c) = make_uint2(u.x, u.y);
+        *reinterpret_cast<uint2*>(Sl + r * ldv + c) = make_uint2(u.z, u.w);
+      }
+      __syncthreads();
+      if (!active) continue;
+      for (int ks = 0; ks < rows; ks += 16) {
+        uint32_t ah[4], al[4];
+        load_a_frag(ah, Qh, ldq, r0, ds + ks, lane);
+        load_a_frag(al, Ql, ldq, r0, ds + ks, lane);
+#pragma unroll
+        for (int i = 0; i < NT; ++i)
+          if (n_base + 8 * i < e) {
+            uint32_t bh[2], bl[2];
+            load_b_frag_kn(bh, Sh, ldv, ks, n_base + 8 * i, lane);
+            load_b_frag_kn(bl, Sl, ldv, ks, n_base + 8 * i, lane);
+            mma_bf16_16816(acc[i], ah, bh);
+            mma_bf16_16816(acc[i], al, bh);
+            mma_bf16_16816(acc[i], ah, bl);
+          }
+      }
+    }
+    const float f_lo = rc_power(lg, r0 + g + 1), f_hi = rc_power(lg, r0 + g + 9);
+#pragma unroll
+    for (int i = 0; i < NT; ++i) {
+      acc[i][0] *= f_lo, acc[i][1] *= f_lo;
+      acc[i][2] *= f_hi, acc[i][3] *= f_hi;
+    }
+  }
+  if (active) {
+#pragma unroll
+    for (int kk = 0; kk < 4; ++kk)
+      if (kk <= rg) {
+#pragma unroll
+        for (int i = 0; i < NT; ++i)
+          if (n_base + 8 * i < e) {
+            uint32_t b[2];
+            load_b_frag_kn(b, V, ldv, kk * 16, n_base + 8 * i, lane);
+            mma_bf16_16816(acc[i], ph[kk], b);
+            mma_bf16_16816(acc[i], pl[kk], b);
+          }
+      }
+    float s_lo = 0.f, s_hi = 0.f;
+#pragma unroll
+    for (int i = 0; i < NT; ++i)
+      if (n_base + 8 * i < e) {
+        s_lo += acc[i][0] * acc[i][0] + acc[i][1] * acc[i][1];
+        s_hi += acc[i][2] * acc[i][2] + acc[i][3] * acc[i][3];
+      }
+#pragma unroll
+    for (int o = 1; o < 4; o <<= 1) {
+      s_lo += __shfl_xor_sync(0xffffffffu, s_lo, o);
+      s_hi += __shfl_xor_sync(0xffffffffu, s_hi, o);
+    }
+    if (t == 0) row_ss[warp >> 2][r0 + g] = s_lo, row_ss[warp >> 2][r0 + g + 8] = s_hi;
+  }
+  __syncthreads();
+  if (!active) return;
+#pragma unroll
+  for (int half = 0; half < 2; ++half) {
+    const int r = r0 + g + 8 * half;
+    if (r >= n) continue;
+    const float f = 1.f / sqrtf((row_ss[0][r] + row_ss[1][r]) / static_cast<float>(e) + p.eps);
+    const long long tok = t0 + r;
+    const __nv_bfloat16* gr = p.gate + tok * p.ldg + h * e;
+    __nv_bfloat16* o = p.out + (tok * p.H + h) * e;
+#pragma unroll
+    for (int i = 0; i < NT; ++i) {
+      const int c = n_base + 8 * i + 2 * t;
+      if (n_base + 8 * i < e) {
+        const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gr + c));
+        const float a0 = (p.gate_sigmoid ? 1.f : z.x) / (1.f + expf(-z.x)), a1 = (p.gate_sigmoid ? 1.f : z.y) / (1.f + expf(-z.y));
+        *reinterpret_cast<__nv_bfloat162*>(o + c) = __floats2bfloat162_rn(acc[i][2 * half] * f * a0, acc[i][2 * half + 1] * f * a1);
+      }
+    }
+  }
+}
+
+static size_t rc_sum_smem(int d, int e) { return sizeof(__nv_bfloat16) * kRcTokens * (2 * static_cast<size_t>(d + 8) + (e + 8)); }
+static size_t rc_output_smem(int d, int e) {
+  return sizeof(__nv_bfloat16) * kRcTokens * (2 * static_cast<size_t>(d + 8) + (e + 8) + 2 * static_cast<size_t>((d > e ? d : e) + 8));
+}
+
+template <int NT>
+static int launch_retention_output(const RetentionChunkParams& p, int chunks, cudaStream_t s) {
+  const size_t smem = rc_output_smem(p.d, p.e);
+  auto kern = retention_chunk_output_kernel<NT>;
+  LLMCTL_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
+  kern<<<dim3(chunks, p.nh), 256, smem, s>>>(p);
+  return 0;
+}
+
 }  // namespace llmctl
 
 using namespace llmctl;
@@ -127,5 +499,43 @@ LLMCTL_API int llmctl_retention_step(const void* q, long long ldq, const void* k
   int rc = 0;
   LLMCTL_DISPATCH_DTYPE(is_fp32, T, (rc = dispatch_matrix_step<T, 3>(p, nportions, (cudaStream_t)stream)));
   if (rc) return rc;
+  LLMCTL_RETURN_LAST();
+}
+
+// 1 when bf16 prompts of these sizes run in chunks: d and e multiples of 16 up to 256, pairs in groups of four.
+LLMCTL_API int llmctl_retention_chunked_ok(int d, int e, int rot) {
+  return (d > 0 && e > 0 && d % 16 == 0 && e % 16 == 0 && d <= 256 && e <= 256 && rot % 8 == 0 && rot <= d && rc_output_smem(d, e) <= 220 * 1024) ? 1 : 0;
+}
+
+// bf16 only; rows of q, k, v and gate start at 16-byte boundaries.  tiles: the 64-token tiles of all portions, in order; cs: fp32
+// scratch [tokens, rot]; scratch: fp32 [chunks, heads_per_pass, d, e].  out: [tokens, H e], normed and gated.
+LLMCTL_API int llmctl_retention_chunked(const void* q, long long ldq, const void* k, long long ldk, const void* v, long long ldv,
+                                        const int* positions, const float* freq, int rot, const float* decay_m1, const int* portions,
+                                        int nportions, const int* tiles, int chunks, int tokens, float* state, const void* gate, long long ldg,
+                                        int gate_kind, float eps, float* cs, float* scratch, int heads_per_pass, void* out, int H, int d, int e,
+                                        void* stream) {
+  LLMCTL_BEGIN();
+  LLMCTL_REQUIRE(llmctl_retention_chunked_ok(d, e, rot) && H > 0 && heads_per_pass > 0 && decay_m1 && scratch && (rot == 0 || (freq && cs)));
+  LLMCTL_REQUIRE(((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v) | reinterpret_cast<uintptr_t>(gate) |
+                   reinterpret_cast<uintptr_t>(state) | reinterpret_cast<uintptr_t>(scratch) | reinterpret_cast<uintptr_t>(cs) | reinterpret_cast<uintptr_t>(out)) & 15) == 0 &&
+                 ldq % 8 == 0 && ldk % 8 == 0 && ldv % 8 == 0 && ldg % 8 == 0);
+  if (chunks == 0 || tokens == 0) return 0;
+  cudaStream_t s = (cudaStream_t)stream;
+  RetentionChunkParams p{(const __nv_bfloat16*)q, (const __nv_bfloat16*)k, (const __nv_bfloat16*)v, (const __nv_bfloat16*)gate, ldq, ldk, ldv, ldg,
+                         (const float2*)cs, rot / 2, decay_m1, portions, nportions, tiles, state, scratch, (__nv_bfloat16*)out, H, d, e, 0, 0,
+                         gate_kind, eps};
+  if (rot > 0) retention_angles_kernel<<<(tokens * (rot / 2) + 255) / 256, 256, 0, s>>>(positions, freq, rot / 2, (float2*)cs, tokens);
+  const size_t smem = rc_sum_smem(d, e);
+  LLMCTL_CHECK(cudaFuncSetAttribute(retention_chunk_sum_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
+  for (int h0 = 0; h0 < H; h0 += heads_per_pass) {
+    p.h0 = h0;
+    p.nh = H - h0 < heads_per_pass ? H - h0 : heads_per_pass;
+    retention_chunk_sum_kernel<<<dim3(chunks, p.nh), 256, smem, s>>>(p);
+    retention_chunk_chain_kernel<<<dim3(nportions, p.nh, (d * e / 4 + 255) / 256), 256, 0, s>>>(p);
+    const int nt = (e / 8 + 1) / 2;
+    const int rc = nt <= 2 ? launch_retention_output<2>(p, chunks, s) : nt <= 4 ? launch_retention_output<4>(p, chunks, s)
+                 : nt <= 8 ? launch_retention_output<8>(p, chunks, s) : launch_retention_output<16>(p, chunks, s);
+    if (rc) return rc;
+  }
   LLMCTL_RETURN_LAST();
 }

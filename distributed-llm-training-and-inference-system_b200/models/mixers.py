@@ -214,7 +214,9 @@ class LatentAttention(nn.Module):
                                    self.rot_freq, self.rot_mult, s.scale, hpt, batch.max_context,
                                    batch.attention_splits(s.heads, rows, span), rows=rows, sinks=self.sink, window=s.window,
                                    head_gate=d[:, self.gate_at:self.gate_at + s.heads] if s.head_gate else None)
-        o = torch.bmm(ol.transpose(0, 1), self.w_uv.transpose(1, 2)).transpose(0, 1).reshape(T, s.heads * s.vdim)
+        o = torch.empty(T, s.heads * s.vdim, dtype=ol.dtype, device=ol.device)          # the product lands head by head in place
+        with torch.no_grad():
+            torch.bmm(ol.transpose(0, 1), self.w_uv.transpose(1, 2), out=o.view(T, s.heads, s.vdim).transpose(0, 1))
         if s.out_gate:
             o = sigmoid_gate_(o, d[:, self.gate_at:self.gate_at + s.heads * s.vdim])
         return ops.linear(o, self.w_o)
@@ -821,7 +823,7 @@ class Retention(nn.Module):
         p = ops.linear(h, self.w_in)
         q, k, v, g = (p[:, a:b] for a, b in self.at.values())
         y = retops.retention(q, k, v, g, batch.positions, self.rot_freq, s.rot_dims, self.decay_m1, batch.portions, state[0], s.heads, s.dim,
-                             s.vdim, self.eps, decode=batch.decode_only)
+                             s.vdim, self.eps, decode=batch.decode_only, tiles=batch.tiles(retops.CHUNK))
         return ops.linear(y, self.w_o)
 
 

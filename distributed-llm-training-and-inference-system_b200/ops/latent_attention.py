@@ -36,7 +36,8 @@ WINDOW_ALIGN = 32           # a window's first key tile starts at a multiple of 
 ROWS_PER_TILE = 16          # query rows (token, head) a CTA owns; tiles are built by the engine with this limit
 ROWS_PER_TILE_WIDE = 32     # the tensor-core kernel also takes tiles of 32 rows (half the key traffic per row)
 ROWS_PER_TILE_TCGEN05 = 128     # query rows per CTA of the tcgen05 kernel (UMMA M)
-TILE_WIDTHS = (ROWS_PER_TILE, ROWS_PER_TILE_WIDE, ROWS_PER_TILE_TCGEN05)
+ROWS_PER_TILE_CHUNK = 64        # tokens of a retention chunk (ops/retention.py)
+TILE_WIDTHS = (ROWS_PER_TILE, ROWS_PER_TILE_WIDE, ROWS_PER_TILE_CHUNK, ROWS_PER_TILE_TCGEN05)
 
 
 def uses_tensor_cores(dtype: torch.dtype, R: int, dr: int) -> bool:

@@ -1,9 +1,10 @@
-"""Serving throughput of a ragged-batch design (Nafazen, Teluzen, Namisun, Tupidra, Zokepel) beside the GPT/LLaMA family at equal parameter count:
+"""Serving throughput of a ragged-batch design (Nafazen, Teluzen, Namisun, Tupidra, Zokepel, Kozasun) beside the GPT/LLaMA family at equal parameter count:
 prefill and decode tokens/s through ``InferenceEngine.generate`` (the scheduler, block manager and step function a
 user gets), random weights, a few layer sizes that resemble real models; plus device-timed runs of the design's own
 attention and expert kernels against the measured roofline, next to the GPT family's like kernels.
-``bench.py --arch-compare nafazen|teluzen|namisun|tupidra|zokepel`` prints the result as one JSON line.  Tupidra and Zokepel are
-also set beside Namisun (another parallel-layout design with state slots) of equal width and depth, with both designs' like kernels.
+``bench.py --arch-compare nafazen|teluzen|namisun|tupidra|zokepel|kozasun`` prints the result as one JSON line.  Tupidra and Zokepel are
+also set beside Namisun (another parallel-layout design with state slots) of equal width and depth, Kozasun beside Zokepel, with both
+designs' like kernels.
 
 Reference: the reference's serving benchmark is ``llmctl bench e2e`` (reference llmctl/cli/commands/bench.py:98-160)."""
 from __future__ import annotations
@@ -76,6 +77,21 @@ ZOKEPEL_SIZES: Dict[str, Dict[str, Any]] = {
     "w4096": dict(width=4096, vocab=32000, pattern="CDPCDP", ff="1", loop=None, heads=32, kv_heads=32, dim=128, vdim=128, conv=4, decay_rank=128,
                   gate_rank=128, att_heads=32, att_kv_heads=8, att_dim=128, att_vdim=128, bias_rows=32, bias_max=256.0, q_temp=(0.1, 1024),
                   mix_heads=64, mix_dim=64, mix_rank=128, ff_size=12288, limit=7.0),
+}
+
+
+KOZASUN_SIZES: Dict[str, Dict[str, Any]] = {
+    # 6 layers: windowed latent attention, chunked attention, retention, twice; dense and mixture feed-forwards in turn, each kind
+    # once per mixer; four streams
+    "w1024": dict(width=1024, vocab=32000, pattern="LARLAR", ff="DM", streams=4, heads=8, kv_heads=2, dim=128, vdim=128, rot_dims=64, rot_base=20000.0,
+                  chunk=1024, ret_heads=8, ret_dim=128, ret_vdim=128, ret_rot=128, lat_heads=8, lat_dim=128, lat_vdim=128, kv_rank=512, window=512,
+                  ff_size=4096, experts=16, top=4, groups=(4, 2), expert_ff=512, shared_ff=1024),
+    "w2048": dict(width=2048, vocab=32000, pattern="LARLAR", ff="DM", streams=4, heads=16, kv_heads=4, dim=128, vdim=128, rot_dims=64, rot_base=20000.0,
+                  chunk=1024, ret_heads=16, ret_dim=128, ret_vdim=128, ret_rot=128, lat_heads=16, lat_dim=128, lat_vdim=128, kv_rank=512, window=512,
+                  ff_size=8192, experts=16, top=4, groups=(4, 2), expert_ff=1024, shared_ff=2048),
+    "w4096": dict(width=4096, vocab=32000, pattern="LARLAR", ff="DM", streams=4, heads=32, kv_heads=8, dim=128, vdim=128, rot_dims=64, rot_base=20000.0,
+                  chunk=1024, ret_heads=32, ret_dim=128, ret_vdim=128, ret_rot=128, lat_heads=32, lat_dim=128, lat_vdim=128, kv_rank=512, window=512,
+                  ff_size=12288, experts=16, top=4, groups=(4, 2), expert_ff=1024, shared_ff=2048),
 }
 
 
@@ -620,6 +636,143 @@ def _zokepel_kernels(size: Dict[str, Any], peaks: Dict[str, float]) -> Dict[str,
     return res
 
 
+def _kozasun_kernels(size: Dict[str, Any], peaks: Dict[str, float]) -> Dict[str, Any]:
+    """The design's own kernels in isolation (bf16, L2 flushed before every call; prefill 2 x 2048 tokens, decode 32 sequences,
+    context 4096 for the attentions), each next to the like kernel of the closest design at the same sizes: windowed latent
+    attention with head gates against the full-context form; chunked attention with sinks against Zokepel's attention with a
+    bias table over full contexts; projection norms + rotation + append against Zokepel's norms + temperature + append; retention
+    against Zokepel's delta rule and Namisun's gated linear attention; the streams' update + layer norm against Namisun's residual +
+    layer norm; the mixture of experts against Namisun's routing."""
+    from ..ops import elementwise as E
+    from ..ops import hyper_norm as HN
+    from ..ops import latent_attention as L
+    from ..ops import matrix_state as MS
+    from ..ops import moe as M
+    from ..ops import native
+    from ..ops import recurrent as R
+    from ..ops import retention as RT
+    from ..ops import softcap_attention as SA
+    from ..ops import window_attention as WA
+    from ..ops.elementwise import rope_frequencies
+    from .ragged import Portion, RaggedBatch
+    dev = torch.device("cuda")
+    bf = torch.bfloat16
+    W, S = size["width"], size["streams"]
+    H, G, d, e, chunk, rot = size["heads"], size["kv_heads"], size["dim"], size["vdim"], size["chunk"], size["rot_dims"]
+    lH, dn, Rk, window = size["lat_heads"], size["lat_dim"], size["kv_rank"], size["window"]
+    rH, rd, re, rrot = size["ret_heads"], size["ret_dim"], size["ret_vdim"], size["ret_rot"]
+    bs, res = 64, {}
+    Wc = G * (d + e)
+
+    def hbm(key: str, t: float, bytes_: float, **more) -> None:
+        res[key] = {"ms": t * 1e3, "gbs": bytes_ / t / 1e9, "frac_of_hbm": bytes_ / t / 1e9 / peaks["hbm_gbs"], **more}
+
+    def work(flops: float, t: float) -> Dict[str, float]:
+        return {"tflops": flops / t / 1e12, "frac_of_bf16_peak": flops / t / 1e12 / peaks["bf16_tflops"]}
+
+    freq = rope_frequencies(rot, 20000.0)[0].to(dev)
+    sink = torch.randn(H, device=dev)
+    table = SA.bucket_bias_table(torch.randn(32, H), 256.0).to(dev)
+    for name, nseq, ctx, new in (("prefill", 2, 2048, 2048), ("decode", 32, 4096, 1)):
+        per = (ctx + bs - 1) // bs
+        ps = [Portion(i, [0] * new, ctx - new, [], list(range(i * per, (i + 1) * per)), i) for i in range(nseq)]
+        b = RaggedBatch(ps, bs, dev)
+        T = b.num_tokens
+        decode = new == 1
+        # chunked attention
+        cache = torch.randn(nseq * per, bs, Wc, device=dev).to(bf)
+        q = torch.randn(T, H * d, device=dev)
+        width = SA.tile_width(bf, H, G, d, e, True, decode)
+        tile = 1 if decode else width
+        for key, ck, kw in ((f"chunked_attention_{name}", chunk, {}), (f"chunked_attention_full_context_{name}", 0, {}),
+                            (f"zokepel_biased_attention_{name}", 0, dict(table=table))):
+            t = _time_flushed(lambda: SA.softcap_window_attention(q, cache, b.block_tables, b.tiles(width), tile, b.positions, None, None,
+                                                                  None if kw else sink, d ** -0.5, 0.0, 0, 0, H, G, d, e, bs, bf,
+                                                                  max_context=b.max_context, chunk=ck, **kw))
+            pairs = nseq * sum((i % ck if ck else i) + 1 for i in range(ctx - new, ctx))
+            keys = nseq * (ctx if not decode else (((ctx - 1) % ck if ck else ctx - 1) + 1))
+            hbm(key, t, keys * Wc * 2 + T * H * (d * 4 + e * 2), **work(2.0 * H * pairs * (d + e), t))
+        # latent attention
+        lcache = torch.randn(nseq * per, bs, Rk, device=dev).to(bf)
+        ql = torch.randn(lH, T, Rk, device=dev).to(bf).transpose(0, 1)
+        lq, gate = torch.randn(T, lH * dn, device=dev).to(bf), torch.randn(T, lH, device=dev).to(bf)
+        rows = L.ROWS_PER_TILE_TCGEN05 if not decode and L.uses_tcgen05(bf, Rk, 0, bs, True) else L.rows_per_tile(bf, Rk, 0, True, lH if decode else 32)
+        hpt = b.heads_per_tile(lH, rows)
+        for key, win, gt in ((f"window_latent_attention_{name}", window, gate), (f"full_latent_attention_{name}", 0, None)):
+            span = L.key_span(b.max_context, win, rows // hpt)
+            t = _time_flushed(lambda: L.latent_attention(ql, lq, dn, lcache, b.block_tables, b.tiles(rows), b.positions, freq, 1.0, 0.07, hpt, b.max_context,
+                                                         b.attention_splits(lH, rows, span), rows=rows, window=win, head_gate=gt))
+            pairs = nseq * sum(min(i + 1, win) if win else i + 1 for i in range(ctx - new, ctx))
+            keys = nseq * (min(ctx, win) if decode and win else ctx)
+            hbm(key, t, keys * Rk * 2 + T * lH * Rk * 4, **work(2.0 * lH * pairs * 2 * Rk, t))
+        # retention
+        nk, nv = rH * rd, rH * re
+        p = torch.randn(T, 2 * nk + 2 * nv, device=dev).to(bf)
+        rq, rk, rv, rg = p[:, :nk], p[:, nk:2 * nk], p[:, 2 * nk:2 * nk + nv], p[:, 2 * nk + nv:]
+        rfreq, decay = rope_frequencies(rrot, 20000.0)[0].to(dev), -torch.rand(rH, device=dev) * 0.01
+        state = torch.zeros(nseq, rH, rd, re, device=dev)
+        bytes_ = T * 2 * (2 * nk + 3 * nv) + 2 * 4 * state.numel()
+        for key, tl in ((f"retention_{name}", b.tiles(RT.CHUNK)), (f"retention_scan_{name}", None)):
+            t = _time_flushed(lambda: RT.retention(rq, rk, rv, rg, b.positions, rfreq, rrot, decay, b.portions, state, rH, rd, re, 1e-5, decode=decode, tiles=tl))
+            hbm(key, t, bytes_)
+        gz, gzb, gnw = torch.randn(T, nk, device=dev).to(bf), torch.rand(nk, device=dev) * 4, torch.ones(re, device=dev)
+
+        def gla():
+            o = R.gla_scan(rq, rk, rv, gz, gzb, b.portions, state, rH, rd, re, rd ** -0.5, 16.0)
+            return R.gla_output(o, gnw, rg, rH, re, 1e-6, bf)
+        hbm(f"namisun_gla_{name}", _time_flushed(gla), bytes_ + T * 2 * nk)
+        C = 2 * nk + nv
+        conv_w, conv, speed = torch.randn(C, 4, device=dev), torch.zeros(nseq, 3, C, device=dev), torch.rand(rH, device=dev)
+        bb = torch.randn(T, rH, device=dev).to(bf)
+        t = _time_flushed(lambda: MS.delta_rule(p[:, :C], conv_w, bb, speed - 4.0, speed, bb, rg, gnw, b.portions, b.seq_rows, state, conv, rH, rH, rd, re,
+                                                False, 1e-6, "silu", decode=decode))
+        hbm(f"zokepel_delta_{name}", t, bytes_ + T * 4 * rH + 2 * 4 * conv.numel())
+        # streams: update + layer norm; one fp32 stream's update + layer norm
+        x, y = torch.randn(T, S, W, device=dev), torch.randn(T, W, device=dev).to(bf)
+        y32, w1, b1 = torch.randn(T, W, device=dev), torch.ones(W, device=dev), torch.zeros(W, device=dev)
+        sw = HN.StreamWeights(torch.rand(S, device=dev), torch.rand(S, device=dev), torch.eye(S, device=dev))
+        t = _time_flushed(lambda: HN.hyper_step(x, y, sw, HN.NextNorm(sw.a, w1, b1), 1e-5, bf))
+        hbm(f"hyper_step_{name}", t, T * W * (8 * S + 2 + 2))
+        t = _time_flushed(lambda: HN.hyper_step(x, y32, sw, HN.NextNorm(sw.a, w1, b1, True), 1e-5, bf))
+        hbm(f"hyper_step_fp32_{name}", t, T * W * (8 * S + 4 + 2 + 4))
+        x1 = torch.randn(T, W, device=dev)
+        t = _time_flushed(lambda: E.parallel_residual(y, y32, x1, 0.5, 1e-5, bf, w1, b1, want_fp32=True))
+        hbm(f"namisun_residual_norm_{name}", t, T * W * (2 + 4 + 4 + 4 + 2 + 4))
+        if not decode:
+            tab, toks = torch.randn(32000, W, device=dev).to(bf), torch.randint(0, 32000, (T,), device=dev)
+            hbm("hyper_embed_prefill", _time_flushed(lambda: HN.hyper_embed(toks, tab, 0.5, S, HN.NextNorm(sw.a, w1, b1), 1e-5)), T * W * (2 + 4 * S + 2))
+            hbm("tupidra_embed_prefill", _time_flushed(lambda: E.embed_scale(toks, tab, 1.0)), T * W * 8)
+            proj, bias = torch.randn(T, H * d + Wc, device=dev).to(bf), torch.randn(H * d + Wc, device=dev)
+            qn, kn = torch.ones(H * d, device=dev), torch.ones(G * d, device=dev)
+            bytes_ = T * ((H * d + Wc) * 2 + H * d * 4 + Wc * 2)
+            t = _time_flushed(lambda: WA.window_qkv_write(proj, bias, qn, kn, H, G, d, e, rot, freq, 1.0, 1e-5, b.positions, b.slots, cache, bs, rot_half=True))
+            hbm("norm_rotate_kv_append_prefill", t, bytes_)
+            t = _time_flushed(lambda: SA.window_kv_append(proj, None, H, G, d, e, False, 1e-6, b.slots, cache, qk_norm=True, q_temp=(0.1, 1024),
+                                                          positions=b.positions))
+            hbm("zokepel_norm_temp_kv_append_prefill", t, bytes_)
+            dproj = torch.randn(T, Rk + lH * dn + 8, device=dev).to(bf)
+            kvw = torch.ones(Rk, device=dev).to(bf)
+            t = _time_flushed(lambda: L.latent_kv_write(dproj, 0, Rk, 0, None, kvw, lcache, b.slots, b.positions, freq, 1.0, 1e-5))
+            hbm("latent_kv_write_prefill", t, T * Rk * 4)
+            F = size["ff_size"]
+            gu = torch.randn(T, 2 * F, device=dev).to(bf)
+            hbm("gated_gelu_prefill", _time_flushed(lambda: E.gated_gelu_tanh(gu)), T * F * 6)
+    E_, top, F = size["experts"], size["top"], size["expert_ff"]
+    for T in (4096, 32):
+        x = torch.randn(T, W, device=dev)
+        wr, corr = (torch.randn(E_, W, device=dev) / W ** 0.5).to(bf), torch.randn(E_, device=dev) * 0.01
+        wgu = (torch.randn(E_, 2 * F, W, device=dev) / W ** 0.5).to(bf)
+        wd = (torch.randn(E_, W, F, device=dev) / F ** 0.5).to(bf)
+        for key, kw in ((f"moe_ffn_{T}_tokens", dict(group_best=2, weight_scale=2.0)), (f"namisun_routing_moe_ffn_{T}_tokens", dict(softmax=True, renormalise=True))):
+            t = _time_flushed(lambda: M.moe_ffn(x, bf, wr, wgu, wd, top, scale_input=False, correction=corr, groups=size["groups"], **kw))
+            hbm(key, t, 6.0 * E_ * F * W + T * W * 8, **work(2.0 * T * top * 3 * F * W, t))
+            t = _time_flushed(lambda: M.route(x, wr, top, correction=corr, groups=size["groups"], **kw))
+            res[key]["route_ms"] = t * 1e3
+    res.update(_gpt_kernels(size, peaks))
+    res["native_launches"] = native.launch_count
+    return res
+
+
 def _gpt_kernels(size: Dict[str, Any], peaks: Dict[str, float]) -> Dict[str, Any]:
     """The GPT family's like kernels at like sizes: causal flash attention over the same 2 x 2048 tokens, paged decode
     attention over the same 32 contexts of 4096 (head size 128 for both), and the SwiGLU feed-forward's two GEMMs on
@@ -669,6 +822,9 @@ def run(which: str = "nafazen", sizes: List[str] | None = None, prompt_len: int 
     elif which == "zokepel":
         from ..models.zokepel import ZokepelConfig as Config, example_config
         table, kernels = ZOKEPEL_SIZES, _zokepel_kernels
+    elif which == "kozasun":
+        from ..models.kozasun import KozasunConfig as Config, example_config
+        table, kernels = KOZASUN_SIZES, _kozasun_kernels
     else:
         raise ValueError(f"no architecture comparison for {which!r}")
     peaks = _peaks()
@@ -690,6 +846,11 @@ def run(which: str = "nafazen", sizes: List[str] | None = None, prompt_len: int 
             ccfg = NamisunConfig.from_dict(namisun_example(**NAMISUN_SIZES[name]), name=f"namisun-{name}")
             row["namisun_params"] = ccfg.num_parameters()
             row["namisun"] = _serve(ccfg, prompts, new_tokens, 64)
+        if which == "kozasun" and name in ZOKEPEL_SIZES:                        # the closest design: matrix states beside paged attention
+            from ..models.zokepel import ZokepelConfig, example_config as zokepel_example
+            ccfg = ZokepelConfig.from_dict(zokepel_example(**ZOKEPEL_SIZES[name]), name=f"zokepel-{name}")
+            row["zokepel_params"] = ccfg.num_parameters()
+            row["zokepel"] = _serve(ccfg, prompts, new_tokens, 64)
         row["seconds"] = round(time.time() - t0, 1)
         out["sizes"][name] = row
     return out

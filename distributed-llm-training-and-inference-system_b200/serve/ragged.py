@@ -39,7 +39,7 @@ class RaggedBatch:
                  pad_to: Optional[Tuple[int, int, int]] = None):
         self.block_size, self.device, self._sms, self.pad_to = block_size, device, sm_count, pad_to
         self.decode_only = all(len(p.tokens) == 1 for p in portions)
-        # attention query tiles come in the widths the kernels take (16 / 32 / 128 rows); a tile of a decode-only batch
+        # token tiles come in the widths the kernels take (attention 16 / 32 / 128 rows, retention 64 tokens); a tile of a decode-only batch
         # is one token with as many of its heads as fit
         self._tile_tokens = tuple(1 if self.decode_only else w for w in TILE_WIDTHS)
         if pad_to is not None:

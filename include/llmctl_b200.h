@@ -424,6 +424,14 @@ int llmctl_retention_step(const void* q, long long ldq, const void* k, long long
                           int nportions, float* state, const void* gate, long long ldg, int gate_kind, float eps, void* out, int H,
                           int d, int e, int is_fp32, void* stream);
 
+/* bf16 prompts in chunks of 64 tokens on the tensor cores, head norm and gate included (see the source for the buffers). */
+int llmctl_retention_chunked_ok(int d, int e, int rot);
+int llmctl_retention_chunked(const void* q, long long ldq, const void* k, long long ldk, const void* v, long long ldv,
+                             const int* positions, const float* freq, int rot, const float* decay_m1, const int* portions,
+                             int nportions, const int* tiles, int chunks, int tokens, float* state, const void* gate, long long ldg,
+                             int gate_kind, float eps, float* cs, float* scratch, int heads_per_pass, void* out, int H, int d, int e,
+                             void* stream);
+
 #ifdef __cplusplus
 }
 #endif
