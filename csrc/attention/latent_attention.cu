@@ -246,14 +246,14 @@ latent_attention_merge_kernel(const float* __restrict__ partial, T* __restrict__
     float gm = -INFINITY;
     for (int s = threadIdx.x; s < nsplit; s += 32) gm = fmaxf(gm, p[s * (R + 2) + R]);
     gm = warp_max(gm);
+    float gl = 0.f;
     for (int s = threadIdx.x; s < nsplit; s += 32) {
       const float ms = p[s * (R + 2) + R];
       wsplit[s] = ms != -INFINITY ? expf(ms - gm) : 0.f;
+      gl += p[s * (R + 2) + R + 1] * wsplit[s];
     }
-    __syncwarp();
+    gl = warp_sum(gl);
     if (threadIdx.x == 0) {
-      float gl = 0.f;
-      for (int s = 0; s < nsplit; ++s) gl += p[s * (R + 2) + R + 1] * wsplit[s];
       s_inv = (gl > 0.f ? 1.f / gl : 0.f) * latent_head_gate(head_gate, gate_ld, base / H, static_cast<int>(base % H));
     }
   }
@@ -261,6 +261,7 @@ latent_attention_merge_kernel(const float* __restrict__ partial, T* __restrict__
   const float inv = s_inv;
   for (int c = threadIdx.x; c < R; c += blockDim.x) {
     float a = 0.f;
+#pragma unroll 8
     for (int s = 0; s < nsplit; ++s) a += p[s * (R + 2) + c] * wsplit[s];
     out[base * R + c] = from_f32<T>(a * inv);
   }
@@ -380,14 +381,21 @@ latent_attention_tc_kernel(const TQ* __restrict__ ql, long long ql_st, long long
   const int k_begin = latent_first_key(row_pos[0], window) + split * keys_per_split;
   const int k_end = min(last + 1, k_begin + keys_per_split);
   const int vec_per_row = D >> 3;
+  // cache rows of a tile's keys are looked up (page table) one tile ahead of the copies that use them
+  __shared__ long long rowoff[2][kTcKeys];
+  auto index_tile = [&](int j0, int which) {
+    if (tid < kTcKeys) {
+      const int j = j0 + tid;
+      rowoff[which][tid] = j < k_end ? (static_cast<long long>(bt[j / block_size]) * block_size + (j % block_size)) * D : -1;
+    }
+  };
   // a warp per key row, asynchronous 16-byte copies of the cache rows as they are
-  auto load_tile = [&](int j0, __nv_bfloat16* Kd) {
+  auto load_tile = [&](int which, __nv_bfloat16* Kd) {
     for (int jj = warp; jj < kTcKeys; jj += kWarps) {
-      const int j = j0 + jj;
       __nv_bfloat16* dst = Kd + jj * Dp;
-      if (j < k_end) {
-        const long long slot = static_cast<long long>(bt[j / block_size]) * block_size + (j % block_size);
-        const __nv_bfloat16* src = cache + slot * D;
+      const long long off = rowoff[which][jj];
+      if (off >= 0) {
+        const __nv_bfloat16* src = cache + off;
         for (int v = lane; v < vec_per_row; v += 32) cp_async_16(dst + v * 8, src + v * 8);
       } else {
         for (int v = lane; v < vec_per_row; v += 32) *reinterpret_cast<uint4*>(dst + v * 8) = make_uint4(0u, 0u, 0u, 0u);
@@ -396,24 +404,29 @@ latent_attention_tc_kernel(const TQ* __restrict__ ql, long long ql_st, long long
     cp_async_commit();
   };
   // With two stages the copy of tile i + 1 is in flight while tile i is multiplied.
-  int buf = 0;
-  if (stages == 2 && k_begin < k_end) load_tile(k_begin, Ks0);
+  int buf = 0, odd = 0;
+  index_tile(k_begin, 0);
+  index_tile(k_begin + kTcKeys, 1);
+  __syncthreads();
+  if (stages == 2 && k_begin < k_end) load_tile(0, Ks0);
   for (int j0 = k_begin; j0 < k_end; j0 += kTcKeys) {
     __nv_bfloat16* Ks = Ks0 + buf * kTcKeys * Dp;
     __syncthreads();                       // the previous tile's products are done: its buffer may be overwritten
     if (stages == 2) {
       if (j0 + kTcKeys < k_end) {
-        load_tile(j0 + kTcKeys, Ks0 + (buf ^ 1) * kTcKeys * Dp);
+        load_tile(odd ^ 1, Ks0 + (buf ^ 1) * kTcKeys * Dp);
         cp_async_wait_prior();
       } else {
         cp_async_wait_all();
       }
       buf ^= 1;
     } else {
-      load_tile(j0, Ks);
+      load_tile(odd, Ks);
       cp_async_wait_all();
     }
     __syncthreads();
+    index_tile(j0 + 2 * kTcKeys, odd);     // its last readers ran before this barrier, its next ones run after another
+    odd ^= 1;
     {
       float sacc[2][4] = {};                   // two independent accumulation chains over alternate k-steps
       int k0 = 0;
@@ -519,7 +532,7 @@ static size_t latent_attention_tc_smem(int R, int dr, int rows, int stages = 1) 
 
 static bool latent_attention_tc_ok(int R, int dr, int rows = kRows) {
   const int D = R + dr;
-  return D % 16 == 0 && R % 8 == 0 && R <= 512 && (rows == 16 || rows == 32) && latent_attention_tc_smem(R, dr, rows) <= 227 * 1024;
+  return D % 16 == 0 && R % 8 == 0 && R <= 512 && (rows == 16 || rows == 32) && latent_attention_tc_smem(R, dr, rows) <= 225 * 1024;      // 1 KB of static shared memory comes on top
 }
 
 template <typename TQ>
@@ -533,7 +546,7 @@ static int launch_latent_attention_tc(const TQ* ql, long long ql_st, long long q
   // only while two CTAs still share an SM (they overlap each other's copies anyway); 32-row tiles whenever it fits
   // (up to R + dr = 576 it does).
   const size_t smem2 = latent_attention_tc_smem(R, dr, rows, 2);
-  const int stages = (rows == 32 ? smem2 <= 227 * 1024 : smem2 <= 113 * 1024) ? 2 : 1;
+  const int stages = (rows == 32 ? smem2 <= 225 * 1024 : smem2 <= 111 * 1024) ? 2 : 1;
   const size_t smem = latent_attention_tc_smem(R, dr, rows, stages);
   const int nt = (R + 63) / 64;
   dim3 grid(ntiles, (H + heads_per_tile - 1) / heads_per_tile, splits);

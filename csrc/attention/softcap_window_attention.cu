@@ -335,23 +335,34 @@ softcap_attention_merge_kernel(const SoftcapAttnParams p, int head_blocks) {
   for (int r = threadIdx.x >> 5; r < nrows; r += blockDim.x >> 5) {
     const long long t = t0 + r / HB;
     const int h = hblk * HB + r % HB;
-    float mx = -INFINITY;
-    for (int s = 0; s < p.splits; ++s) mx = fmaxf(mx, p.part_ml[((unit * p.splits + s) * kSwRows + r) * 2]);
-    float ls = 0.f;
-    for (int s = 0; s < p.splits; ++s) {
-      const float* ml = p.part_ml + ((unit * p.splits + s) * kSwRows + r) * 2;
-      if (ml[0] > -INFINITY) ls += ml[1] * expf(ml[0] - mx);
+    float ms[2] = {-INFINITY, -INFINITY}, lw[2] = {0.f, 0.f};              // lane s holds slices s and s + 32 (splits <= 64)
+#pragma unroll
+    for (int k = 0; k < 2; ++k)
+      if (lane + 32 * k < p.splits) {
+        const float2 ml = *reinterpret_cast<const float2*>(p.part_ml + ((unit * p.splits + lane + 32 * k) * kSwRows + r) * 2);
+        ms[k] = ml.x;
+        lw[k] = ml.y;
+      }
+    const float mx = warp_max(fmaxf(ms[0], ms[1]));
+    float w[2];
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+      w[k] = ms[k] > -INFINITY ? expf(ms[k] - mx) : 0.f;
+      lw[k] *= w[k];
     }
+    const float ls = warp_sum(lw[0] + lw[1]);
     const float inv = ls > 0.f ? 1.f / ls : 0.f;
     T* orow = static_cast<T*>(p.out) + (t * H + h) * e;
     const T* grow = p.gate ? static_cast<const T*>(p.gate) + t * p.gate_ld + static_cast<long long>(h) * e : nullptr;
-    for (int c = lane; c < e; c += 32) {
+    for (int c0 = 0; c0 < e; c0 += 32) {
+      const int c = c0 + lane;
       float a = 0.f;
+#pragma unroll 8
       for (int s = 0; s < p.splits; ++s) {
-        const long long row = (unit * p.splits + s) * kSwRows + r;
-        const float mv = p.part_ml[row * 2];
-        if (mv > -INFINITY) a += p.part_o[row * e + c] * expf(mv - mx);
+        const float ws = __shfl_sync(0xffffffffu, s < 32 ? w[0] : w[1], s & 31);
+        if (ws != 0.f && c < e) a += p.part_o[((unit * p.splits + s) * kSwRows + r) * e + c] * ws;      // empty slices wrote sums of 0 weight
       }
+      if (c >= e) continue;
       float o = a * inv;
       if (grow) o *= 1.f / (1.f + expf(-to_f32(grow[c])));
       orow[c] = from_f32<T>(o);
@@ -445,16 +456,20 @@ softcap_attention_mma_kernel(const SoftcapAttnParams p, int decode) {
       rowoff[stage][tid] = j < kt.limit(it) ? (static_cast<long long>(table[j / bs]) * bs + j % bs) * Wc : -1;
     }
   };
+  // 2^sh lanes copy a key's 16-byte chunks (its key numbers, then its value numbers)
+  const int sh = chunks > 16 ? 5 : chunks > 8 ? 4 : 3, sub = lane & ((1 << sh) - 1);
   auto load_tile = [&](int stage) {
-    for (int i = tid; i < kSwKT * chunks; i += nthreads) {
-      const int kk = i / chunks, ch = i % chunks;
+    for (int kk = tid >> sh; kk < kSwKT; kk += nthreads >> sh) {
       const long long off = rowoff[stage][kk];
-      __nv_bfloat16* dst = ch < kch ? Ks + (stage * kSwKT + kk) * ldk + ch * 8 : Vs + (stage * kSwKT + kk) * ldv + (ch - kch) * 8;
-      if (off >= 0) {
-        const __nv_bfloat16* row = cache + off;
-        cp_async_16(dst, ch < kch ? row + g * d + ch * 8 : row + G * d + g * e + (ch - kch) * 8);
-      } else {
-        *reinterpret_cast<uint4*>(dst) = make_uint4(0u, 0u, 0u, 0u);      // a weight of 0 times stale bits could be a NaN
+      const __nv_bfloat16* krow = cache + off + g * d;
+      const __nv_bfloat16* vrow = cache + off + G * d + g * e - d;        // chunk ch >= kch holds value numbers 8 (ch - kch) ..
+      __nv_bfloat16* kdst = Ks + (stage * kSwKT + kk) * ldk;
+      __nv_bfloat16* vdst = Vs + (stage * kSwKT + kk) * ldv - d;
+      for (int ch = sub; ch < chunks; ch += 1 << sh) {
+        const bool key = ch < kch;
+        __nv_bfloat16* dst = (key ? kdst : vdst) + ch * 8;
+        if (off >= 0) cp_async_16(dst, (key ? krow : vrow) + ch * 8);
+        else *reinterpret_cast<uint4*>(dst) = make_uint4(0u, 0u, 0u, 0u);      // a weight of 0 times stale bits could be a NaN
       }
     }
   };
@@ -744,7 +759,7 @@ LLMCTL_API int llmctl_softcap_window_attention(const float* q, const void* cache
   LLMCTL_REQUIRE(H > 0 && G > 0 && H % G == 0 && d > 0 && e > 0 && e <= 512 && bs > 0 && tile_tokens >= 1 && window >= 0 &&
                  keep_first >= 0 && chunk >= 0 && cap >= 0.f);
   LLMCTL_REQUIRE(table == nullptr || table_len >= 1);
-  LLMCTL_REQUIRE(splits >= 1 && (splits == 1 || (part_ml != nullptr && part_o != nullptr)));
+  LLMCTL_REQUIRE(splits >= 1 && splits <= 64 && (splits == 1 || (part_ml != nullptr && part_o != nullptr)));
   if (ntiles == 0) return 0;
   cudaStream_t s = (cudaStream_t)stream;
   SoftcapAttnParams p{q, cache, block_tables, max_blocks, tiles, positions, gate, gate_ld, slopes, sinks, table, table_len, scale, cap, window, keep_first, chunk,

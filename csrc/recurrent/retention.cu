@@ -103,7 +103,7 @@ struct RetentionChunkParams {
   int nportions;
   const int* tiles;           // [chunks, 4] = (first token row, tokens, portion, 0), portions in order
   float* state;               // [slots, H, d, e]
-  float* scratch;             // [chunks, nh, d, e]: a chunk's sum, then groups of 4 numbers of the state before it as 4 hi, 4 lo
+  float* scratch;             // [chunks, nh, d, e]: a chunk's sum, then groups of 8 numbers of the state before it as 8 hi, 8 lo
   __nv_bfloat16* out;         // [T, H e]
   int H, d, e, h0, nh;        // heads h0 .. h0 + nh - 1
   int gate_sigmoid;
@@ -131,54 +131,97 @@ __device__ __forceinline__ void rc_split4(const float (&v)[4], uint2& hi, uint2&
   lo = make_uint2(pack_bf16x2(r[0], r[1]), pack_bf16x2(r[2], r[3]));
 }
 
-// Rows j of a chunk (x + j ld, d numbers): rotated, times factor * decay^(last - j) (log2_decay 0: no decay), split into hi and lo
-// [64][d + 8] in shared memory; rows past n are zeros.
+// Rows j of a chunk (x + j ld, d numbers): rotated, times factor [* decay^(last - j)], split into hi and lo
+// [64][d + 8] in shared memory; rows past n are zeros.  An item is four pairs or four unrotated numbers; the loads of IT items per
+// thread are in flight together.
+template <int IT, bool DECAY>
 __device__ __forceinline__ void rc_load_rotated(const __nv_bfloat16* x, long long ld, const float2* cs, int half, int d, int n, float factor,
                                                 float log2_decay, int last, __nv_bfloat16* hi, __nv_bfloat16* lo) {
-  const int per = d >> 2, lds = d + 8;
-  for (int i = threadIdx.x; i < kRcTokens * per; i += blockDim.x) {
-    const int j = i / per, c = (i - j * per) << 2;
-    if (c >= half && c < 2 * half) continue;           // the second number of a pair goes with the first
-    float a[4] = {0.f, 0.f, 0.f, 0.f}, b[4] = {0.f, 0.f, 0.f, 0.f};
-    if (j < n) {
-      const float f = factor * rc_power(log2_decay, last - j);
-      load_vec<4>(x + j * ld + c, a);
-      if (c < half) {
-        load_vec<4>(x + j * ld + c + half, b);
-        float w[8];
-        const float* t = reinterpret_cast<const float*>(cs + static_cast<long long>(j) * half + c);
-        *reinterpret_cast<float4*>(w) = *reinterpret_cast<const float4*>(t);
-        *reinterpret_cast<float4*>(w + 4) = *reinterpret_cast<const float4*>(t + 4);
+  const int pairs = half >> 2, per = (d >> 2) - pairs, lds = d + 8, total = kRcTokens * per;
+  const int dj = 256 / per, dk = 256 - dj * per;       // CTAs of 256 threads
+  int i = threadIdx.x, j = i / per, k = i - j * per;
+  while (i < total) {
+    float a[IT][4], b[IT][4], w[IT][8];
+    int jj[IT], cc[IT];
 #pragma unroll
-        for (int k = 0; k < 4; ++k) {
-          const float u = a[k], v = b[k];
-          a[k] = (u * w[2 * k] - v * w[2 * k + 1]) * f;
-          b[k] = (v * w[2 * k] + u * w[2 * k + 1]) * f;
+    for (int u = 0; u < IT; ++u) {
+      jj[u] = i < total ? j : -1;
+      cc[u] = k < pairs ? k << 2 : (k << 2) + half;
+#pragma unroll
+      for (int v = 0; v < 4; ++v) a[u][v] = b[u][v] = 0.f;
+      if (i < total && j < n) {
+        load_vec<4>(x + j * ld + cc[u], a[u]);
+        if (cc[u] < half) {
+          load_vec<4>(x + j * ld + cc[u] + half, b[u]);
+          const float* t = reinterpret_cast<const float*>(cs + static_cast<long long>(j) * half + cc[u]);
+          *reinterpret_cast<float4*>(w[u]) = *reinterpret_cast<const float4*>(t);
+          *reinterpret_cast<float4*>(w[u] + 4) = *reinterpret_cast<const float4*>(t + 4);
+        }
+      }
+      i += 256;
+      j += dj;
+      k += dk;
+      if (k >= per) k -= per, ++j;
+    }
+#pragma unroll
+    for (int u = 0; u < IT; ++u) {
+      const int row = jj[u], c = cc[u];
+      if (row < 0) continue;
+      float f = factor;
+      if (DECAY) f = row < n ? factor * rc_power(log2_decay, last - row) : 0.f;
+      if (c < half && row < n) {
+#pragma unroll
+        for (int v = 0; v < 4; ++v) {
+          const float p = a[u][v], q = b[u][v];
+          a[u][v] = (p * w[u][2 * v] - q * w[u][2 * v + 1]) * f;
+          b[u][v] = (q * w[u][2 * v] + p * w[u][2 * v + 1]) * f;
         }
       } else {
 #pragma unroll
-        for (int k = 0; k < 4; ++k) a[k] *= f;
+        for (int v = 0; v < 4; ++v) a[u][v] *= f;
       }
-    }
-    uint2 h, l;
-    rc_split4(a, h, l);
-    *reinterpret_cast<uint2*>(hi + j * lds + c) = h;
-    *reinterpret_cast<uint2*>(lo + j * lds + c) = l;
-    if (c < half) {
-      rc_split4(b, h, l);
-      *reinterpret_cast<uint2*>(hi + j * lds + c + half) = h;
-      *reinterpret_cast<uint2*>(lo + j * lds + c + half) = l;
+      uint2 h, l;
+      rc_split4(a[u], h, l);
+      *reinterpret_cast<uint2*>(hi + row * lds + c) = h;
+      *reinterpret_cast<uint2*>(lo + row * lds + c) = l;
+      if (c < half) {
+        rc_split4(b[u], h, l);
+        *reinterpret_cast<uint2*>(hi + row * lds + c + half) = h;
+        *reinterpret_cast<uint2*>(lo + row * lds + c + half) = l;
+      }
     }
   }
 }
 
+// asynchronous copies of a chunk's rows (rows past n: zeros); the caller commits and waits
 __device__ __forceinline__ void rc_load_rows(const __nv_bfloat16* x, long long ld, int cols, int n, __nv_bfloat16* dst, int lds) {
-  const int per = cols >> 3;
-  for (int i = threadIdx.x; i < kRcTokens * per; i += blockDim.x) {
-    const int j = i / per, c = (i - j * per) << 3;
-    const uint4 u = j < n ? *reinterpret_cast<const uint4*>(x + j * ld + c) : make_uint4(0u, 0u, 0u, 0u);
-    *reinterpret_cast<uint4*>(dst + j * lds + c) = u;
+  const int per = cols >> 3, dj = 256 / per, dk = 256 - dj * per;
+  int j = threadIdx.x / per, k = threadIdx.x - j * per;
+  for (; j < kRcTokens; j += dj, k += dk) {
+    if (k >= per) {
+      k -= per;
+      if (++j >= kRcTokens) break;
+    }
+    const int c = k << 3;
+    if (j < n) cp_async_16(dst + j * lds + c, x + j * ld + c);
+    else *reinterpret_cast<uint4*>(dst + j * lds + c) = make_uint4(0u, 0u, 0u, 0u);
   }
+}
+
+// two neighbouring B fragments (8 columns each) by one ldmatrix: operand stored [n][k] / [k][n]
+__device__ __forceinline__ void rc_b2_nk(uint32_t (&b)[4], const __nv_bfloat16* m, int ld, int n0, int k0, int lane) {
+  const __nv_bfloat16* p = m + (n0 + (lane & 7) + ((lane >> 4) << 3)) * ld + k0 + (((lane >> 3) & 1) << 3);
+  const uint32_t addr = static_cast<uint32_t>(__cvta_generic_to_shared(p));
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n" : "=r"(b[0]), "=r"(b[1]), "=r"(b[2]), "=r"(b[3]) : "r"(addr));
+}
+__device__ __forceinline__ void rc_b2_kn(uint32_t (&b)[4], const __nv_bfloat16* m, int ld, int k0, int n0, int lane) {
+  const __nv_bfloat16* p = m + (k0 + (lane & 15)) * ld + n0 + ((lane >> 4) << 3);
+  const uint32_t addr = static_cast<uint32_t>(__cvta_generic_to_shared(p));
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];\n" : "=r"(b[0]), "=r"(b[1]), "=r"(b[2]), "=r"(b[3]) : "r"(addr));
+}
+__device__ __forceinline__ void rc_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  const uint32_t b[2] = {b0, b1};
+  mma_bf16_16816(c, a, b);
 }
 
 // A fragment of A[m][k] = s[k0 + k][m0 + m] (operand stored [k][m] row-major): ldmatrix with transposition
@@ -191,7 +234,7 @@ __device__ __forceinline__ void rc_a_frag_km(uint32_t (&a)[4], const __nv_bfloat
 }
 
 // scratch[chunk, head] = sum_j decay^(L-1-j) k_j v_j^T.  Grid: (chunks, heads); a warp owns blocks of 16 x 32 numbers.
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, 3)
 retention_chunk_sum_kernel(const RetentionChunkParams p) {
   extern __shared__ __align__(16) unsigned char rc_smem[];
   const int d = p.d, e = p.e, ldk = d + 8, ldv = e + 8, h = p.h0 + blockIdx.y;
@@ -203,8 +246,10 @@ retention_chunk_sum_kernel(const RetentionChunkParams p) {
   __nv_bfloat16* Kl = Kh + kRcTokens * ldk;
   __nv_bfloat16* V = Kl + kRcTokens * ldk;
   const float lg = rc_log2_decay(p.dm[h]);
-  rc_load_rotated(p.k + t0 * p.ldk + h * d, p.ldk, p.cs + t0 * p.half, p.half, d, n, 1.f / sqrtf(static_cast<float>(d)), lg, n - 1, Kh, Kl);
   rc_load_rows(p.v + t0 * p.ldv + h * e, p.ldv, e, n, V, ldv);
+  cp_async_commit();
+  rc_load_rotated<2, true>(p.k + t0 * p.ldk + h * d, p.ldk, p.cs + t0 * p.half, p.half, d, n, 1.f / sqrtf(static_cast<float>(d)), lg, n - 1, Kh, Kl);
+  cp_async_wait_all();
   __syncthreads();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3;
   const int nb = (e + 31) / 32, blocks = (d / 16) * nb, steps = (n + 15) / 16;
@@ -217,12 +262,14 @@ retention_chunk_sum_kernel(const RetentionChunkParams p) {
       rc_a_frag_km(ah, Kh, ldk, m0, ks * 16, lane);
       rc_a_frag_km(al, Kl, ldk, m0, ks * 16, lane);
 #pragma unroll
-      for (int i = 0; i < 4; ++i)
-        if (n0 + 8 * i < e) {
-          uint32_t bf[2];
-          load_b_frag_kn(bf, V, ldv, ks * 16, n0 + 8 * i, lane);
-          mma_bf16_16816(acc[i], ah, bf);
-          mma_bf16_16816(acc[i], al, bf);
+      for (int i = 0; i < 4; i += 2)
+        if (n0 + 8 * i < e) {                          // e is a multiple of 16
+          uint32_t bf[4];
+          rc_b2_kn(bf, V, ldv, ks * 16, n0 + 8 * i, lane);
+          rc_mma(acc[i], ah, bf[0], bf[1]);
+          rc_mma(acc[i + 1], ah, bf[2], bf[3]);
+          rc_mma(acc[i], al, bf[0], bf[1]);
+          rc_mma(acc[i + 1], al, bf[2], bf[3]);
         }
     }
 #pragma unroll
@@ -235,45 +282,48 @@ retention_chunk_sum_kernel(const RetentionChunkParams p) {
   }
 }
 
-// The chain over a portion's chunks, four numbers of a head's state per thread.  Grid: (portions, heads, d e / 1024).
+// The chain over a portion's chunks, eight numbers of a head's state per thread.  Grid: (portions, heads, d e / 2048).
 __global__ void __launch_bounds__(256)
 retention_chunk_chain_kernel(const RetentionChunkParams p) {
   constexpr int AHEAD = 4;
   const int* pt = p.portions + 4 * blockIdx.x;
   const int n = pt[1], slot = pt[3], h = p.h0 + blockIdx.y;
-  const long long numbers = static_cast<long long>(p.d) * p.e, i = (static_cast<long long>(blockIdx.z) * blockDim.x + threadIdx.x) * 4;
+  const long long numbers = static_cast<long long>(p.d) * p.e, i = (static_cast<long long>(blockIdx.z) * blockDim.x + threadIdx.x) * 8;
   if (n <= 0 || i >= numbers) return;
   int first = 0;
   for (int b = 0; b < static_cast<int>(blockIdx.x); ++b) first += (max(p.portions[4 * b + 1], 0) + kRcTokens - 1) / kRcTokens;
   const int chunks = (n + kRcTokens - 1) / kRcTokens;
   float* st = slot >= 0 ? p.state + (static_cast<long long>(slot) * p.H + h) * numbers + i : nullptr;
-  float4 S = (st && pt[2] > 0) ? *reinterpret_cast<const float4*>(st) : make_float4(0.f, 0.f, 0.f, 0.f);
+  float S[8];
+#pragma unroll
+  for (int k = 0; k < 8; ++k) S[k] = 0.f;
+  if (st && pt[2] > 0) load8_f32(st, S);
   const float lg = log1pf(p.dm[h]);
   const float full = expm1f(lg * kRcTokens), rest = expm1f(lg * static_cast<float>(n - (chunks - 1) * kRcTokens));
   const long long step = static_cast<long long>(p.nh) * numbers;
   float* x = p.scratch + (static_cast<long long>(first) * p.nh + blockIdx.y) * numbers + i;
-  float4 kv[AHEAD];
+  float kv[AHEAD][8];
 #pragma unroll
   for (int a = 0; a < AHEAD; ++a)
-    if (a < chunks) kv[a] = *reinterpret_cast<const float4*>(x + a * step);
+    if (a < chunks) load8_f32(x + a * step, kv[a]);
   for (int c0 = 0; c0 < chunks; c0 += AHEAD) {
 #pragma unroll
     for (int a = 0; a < AHEAD; ++a) {
       const int c = c0 + a;
       if (c >= chunks) break;
-      const float s[4] = {S.x, S.y, S.z, S.w};
-      uint2 hi, lo;
-      rc_split4(s, hi, lo);
+      float r[8];
+#pragma unroll
+      for (int k = 0; k < 8; ++k) r[k] = S[k] - __bfloat162float(__float2bfloat16(S[k]));
+      __nv_bfloat16* pair = reinterpret_cast<__nv_bfloat16*>(x + c * step);       // in place: 8 hi, 8 lo
+      store8_f32(pair, S);
+      store8_f32(pair + 8, r);
       const float gm = c + 1 < chunks ? full : rest;
-      S.x = fmaf(gm, S.x, S.x) + kv[a].x;
-      S.y = fmaf(gm, S.y, S.y) + kv[a].y;
-      S.z = fmaf(gm, S.z, S.z) + kv[a].z;
-      S.w = fmaf(gm, S.w, S.w) + kv[a].w;
-      *reinterpret_cast<uint4*>(x + c * step) = make_uint4(hi.x, hi.y, lo.x, lo.y);
-      if (c + AHEAD < chunks) kv[a] = *reinterpret_cast<const float4*>(x + (c + AHEAD) * step);
+#pragma unroll
+      for (int k = 0; k < 8; ++k) S[k] = fmaf(gm, S[k], S[k]) + kv[a][k];
+      if (c + AHEAD < chunks) load8_f32(x + (c + AHEAD) * step, kv[a]);
     }
   }
-  if (st) *reinterpret_cast<float4*>(st) = S;
+  if (st) store8_f32(st, S);
 }
 
 // Outputs of a chunk and head.  Warp (r, c) = (warp % 4, warp / 4) owns 16 tokens and half of the value columns (NT tiles of 8).
@@ -281,7 +331,7 @@ template <int NT>
 __global__ void __launch_bounds__(256, NT <= 8 ? 2 : 1)
 retention_chunk_output_kernel(const RetentionChunkParams p) {
   extern __shared__ __align__(16) unsigned char rc_smem[];
-  __shared__ float row_ss[2][kRcTokens];
+  __shared__ float row_ss[2][kRcTokens], power[kRcTokens + 1];      // power[i] = decay^i
   const int d = p.d, e = p.e, ldq = d + 8, ldv = e + 8, h = p.h0 + blockIdx.y;
   const int* tile = p.tiles + 4 * blockIdx.x;
   const long long t0 = tile[0];
@@ -292,19 +342,20 @@ retention_chunk_output_kernel(const RetentionChunkParams p) {
   __nv_bfloat16* Qh = reinterpret_cast<__nv_bfloat16*>(rc_smem);
   __nv_bfloat16* Ql = Qh + kRcTokens * ldq;
   __nv_bfloat16* V = Ql + kRcTokens * ldq;
-  __nv_bfloat16* Kh = V + kRcTokens * ldv;             // keys, then 64 rows of the state at a time
+  __nv_bfloat16* Kh = V + kRcTokens * ldv;             // keys, then two stages of 32 rows of the state (hi, lo)
   __nv_bfloat16* Kl = Kh + kRcTokens * ldq;
-  __nv_bfloat16* Sh = Kh;
-  __nv_bfloat16* Sl = Sh + kRcTokens * ldv;
   const float2* cs = p.cs + t0 * p.half;
-  rc_load_rotated(p.q + t0 * p.ldq + h * d, p.ldq, cs, p.half, d, n, 1.f, 0.f, 0, Qh, Ql);
-  rc_load_rotated(p.k + t0 * p.ldk + h * d, p.ldk, cs, p.half, d, n, 1.f / sqrtf(static_cast<float>(d)), 0.f, 0, Kh, Kl);
+  const float lg = rc_log2_decay(p.dm[h]);
+  if (threadIdx.x <= kRcTokens) power[threadIdx.x] = rc_power(lg, threadIdx.x);
   rc_load_rows(p.v + t0 * p.ldv + h * e, p.ldv, e, n, V, ldv);
+  cp_async_commit();
+  rc_load_rotated<4, false>(p.q + t0 * p.ldq + h * d, p.ldq, cs, p.half, d, n, 1.f, 0.f, 0, Qh, Ql);
+  rc_load_rotated<4, false>(p.k + t0 * p.ldk + h * d, p.ldk, cs, p.half, d, n, 1.f / sqrtf(static_cast<float>(d)), 0.f, 0, Kh, Kl);
+  cp_async_wait_all();
   __syncthreads();
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
   const int rg = warp & 3, r0 = rg * 16, n_base = (warp >> 2) * NT * 8;
   const bool active = r0 < n;
-  const float lg = rc_log2_decay(p.dm[h]);
   uint32_t ph[4][4], pl[4][4];                         // decayed scores, A fragments of 16 keys each
   if (active) {
     float s[8][4];
@@ -317,14 +368,17 @@ retention_chunk_output_kernel(const RetentionChunkParams p) {
       load_a_frag(ah, Qh, ldq, r0, ks, lane);
       load_a_frag(al, Ql, ldq, r0, ks, lane);
 #pragma unroll
-      for (int i = 0; i < 8; ++i)
+      for (int i = 0; i < 8; i += 2)
         if (i < 2 * (rg + 1)) {                        // later keys are masked for all rows of the warp
-          uint32_t bh[2], bl[2];
-          load_b_frag_nk(bh, Kh, ldq, 8 * i, ks, lane);
-          load_b_frag_nk(bl, Kl, ldq, 8 * i, ks, lane);
-          mma_bf16_16816(s[i], ah, bh);
-          mma_bf16_16816(s[i], al, bh);
-          mma_bf16_16816(s[i], ah, bl);
+          uint32_t bh[4], bl[4];
+          rc_b2_nk(bh, Kh, ldq, 8 * i, ks, lane);
+          rc_b2_nk(bl, Kl, ldq, 8 * i, ks, lane);
+          rc_mma(s[i], ah, bh[0], bh[1]);
+          rc_mma(s[i + 1], ah, bh[2], bh[3]);
+          rc_mma(s[i], al, bh[0], bh[1]);
+          rc_mma(s[i + 1], al, bh[2], bh[3]);
+          rc_mma(s[i], ah, bl[0], bl[1]);
+          rc_mma(s[i + 1], ah, bl[2], bl[3]);
         }
     }
 #pragma unroll
@@ -332,7 +386,7 @@ retention_chunk_output_kernel(const RetentionChunkParams p) {
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const int dist = r0 + g + (j >> 1) * 8 - (8 * i + 2 * t + (j & 1));
-        s[i][j] = dist >= 0 ? s[i][j] * rc_power(lg, dist) : 0.f;
+        s[i][j] = dist >= 0 ? s[i][j] * power[dist] : 0.f;
       }
 #pragma unroll
     for (int kk = 0; kk < 4; ++kk)
@@ -350,36 +404,63 @@ retention_chunk_output_kernel(const RetentionChunkParams p) {
 #pragma unroll
     for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
   if (has_state) {                                     // uniform over the CTA
-    const uint4* src = reinterpret_cast<const uint4*>(p.scratch + (static_cast<long long>(blockIdx.x) * p.nh + blockIdx.y) * d * e);
-    const int per = e >> 2;
-    for (int ds = 0; ds < d; ds += kRcTokens) {
-      const int rows = min(kRcTokens, d - ds);
-      __syncthreads();                                 // the readers of the keys / the previous rows are done
-      for (int i = tid; i < rows * per; i += 256) {
-        const int r = i / per, c = (i - r * per) << 2;
-        const uint4 u = src[static_cast<long long>(ds + r) * per + (c >> 2)];
-        *reinterpret_cast<uint2*>(Sh + r * ldv + c) = make_uint2(u.x, u.y);
-        *reinterpret_cast<uint2*>(Sl + r * ldv + c) = make_uint2(u.z, u.w);
+    constexpr int SR = kRcTokens / 2;                  // state rows per stage
+    const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(p.scratch + (static_cast<long long>(blockIdx.x) * p.nh + blockIdx.y) * d * e);
+    const int per = e >> 3, slices = (d + SR - 1) / SR;
+    const int dr = 256 / per, dk = 256 - dr * per, first_r = tid / per, first_k = tid - first_r * per;
+    auto fetch = [&](int sl) {                         // rows sl SR .. of the state; 8 hi and 8 lo numbers lie next to each other
+      __nv_bfloat16* Sh = Kh + (sl & 1) * 2 * SR * ldv;
+      const int rows = min(SR, d - sl * SR);
+      int r = first_r, k = first_k;
+      for (; r < rows; r += dr, k += dk) {
+        if (k >= per) {
+          k -= per;
+          if (++r >= rows) break;
+        }
+        const int c = k << 3;
+        const __nv_bfloat16* u = src + (static_cast<long long>(sl * SR + r) * e + c) * 2;
+        cp_async_16(Sh + r * ldv + c, u);
+        cp_async_16(Sh + (SR + r) * ldv + c, u + 8);
       }
-      __syncthreads();
-      if (!active) continue;
-      for (int ks = 0; ks < rows; ks += 16) {
-        uint32_t ah[4], al[4];
-        load_a_frag(ah, Qh, ldq, r0, ds + ks, lane);
-        load_a_frag(al, Ql, ldq, r0, ds + ks, lane);
+    };
+    __syncthreads();                                   // the readers of the keys are done
+    fetch(0);
+    cp_async_commit();
+    if (slices > 1) fetch(1);
+    cp_async_commit();
+    for (int sl = 0; sl < slices; ++sl) {
+      cp_async_wait_prior();
+      __syncthreads();                                 // slice sl has landed
+      const __nv_bfloat16* Sh = Kh + (sl & 1) * 2 * SR * ldv;
+      const __nv_bfloat16* Sl = Sh + SR * ldv;
+      const int rows = min(SR, d - sl * SR);
+      if (active) {
+        for (int ks = 0; ks < rows; ks += 16) {
+          uint32_t ah[4], al[4];
+          load_a_frag(ah, Qh, ldq, r0, sl * SR + ks, lane);
+          load_a_frag(al, Ql, ldq, r0, sl * SR + ks, lane);
 #pragma unroll
-        for (int i = 0; i < NT; ++i)
-          if (n_base + 8 * i < e) {
-            uint32_t bh[2], bl[2];
-            load_b_frag_kn(bh, Sh, ldv, ks, n_base + 8 * i, lane);
-            load_b_frag_kn(bl, Sl, ldv, ks, n_base + 8 * i, lane);
-            mma_bf16_16816(acc[i], ah, bh);
-            mma_bf16_16816(acc[i], al, bh);
-            mma_bf16_16816(acc[i], ah, bl);
-          }
+          for (int i = 0; i < NT; i += 2)
+            if (n_base + 8 * i < e) {
+              uint32_t bh[4], bl[4];
+              rc_b2_kn(bh, Sh, ldv, ks, n_base + 8 * i, lane);
+              rc_b2_kn(bl, Sl, ldv, ks, n_base + 8 * i, lane);
+              rc_mma(acc[i], ah, bh[0], bh[1]);
+              rc_mma(acc[i + 1], ah, bh[2], bh[3]);
+              rc_mma(acc[i], al, bh[0], bh[1]);
+              rc_mma(acc[i + 1], al, bh[2], bh[3]);
+              rc_mma(acc[i], ah, bl[0], bl[1]);
+              rc_mma(acc[i + 1], ah, bl[2], bl[3]);
+            }
+        }
       }
+      if (sl + 2 < slices) {
+        __syncthreads();                               // its readers are done: the stage may be overwritten
+        fetch(sl + 2);
+      }
+      cp_async_commit();
     }
-    const float f_lo = rc_power(lg, r0 + g + 1), f_hi = rc_power(lg, r0 + g + 9);
+    const float f_lo = power[r0 + g + 1], f_hi = power[r0 + g + 9];
 #pragma unroll
     for (int i = 0; i < NT; ++i) {
       acc[i][0] *= f_lo, acc[i][1] *= f_lo;
@@ -391,12 +472,14 @@ retention_chunk_output_kernel(const RetentionChunkParams p) {
     for (int kk = 0; kk < 4; ++kk)
       if (kk <= rg) {
 #pragma unroll
-        for (int i = 0; i < NT; ++i)
+        for (int i = 0; i < NT; i += 2)
           if (n_base + 8 * i < e) {
-            uint32_t b[2];
-            load_b_frag_kn(b, V, ldv, kk * 16, n_base + 8 * i, lane);
-            mma_bf16_16816(acc[i], ph[kk], b);
-            mma_bf16_16816(acc[i], pl[kk], b);
+            uint32_t b[4];
+            rc_b2_kn(b, V, ldv, kk * 16, n_base + 8 * i, lane);
+            rc_mma(acc[i], ph[kk], b[0], b[1]);
+            rc_mma(acc[i + 1], ph[kk], b[2], b[3]);
+            rc_mma(acc[i], pl[kk], b[0], b[1]);
+            rc_mma(acc[i + 1], pl[kk], b[2], b[3]);
           }
       }
     float s_lo = 0.f, s_hi = 0.f;
@@ -428,7 +511,9 @@ retention_chunk_output_kernel(const RetentionChunkParams p) {
       const int c = n_base + 8 * i + 2 * t;
       if (n_base + 8 * i < e) {
         const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gr + c));
-        const float a0 = (p.gate_sigmoid ? 1.f : z.x) / (1.f + expf(-z.x)), a1 = (p.gate_sigmoid ? 1.f : z.y) / (1.f + expf(-z.y));
+        // bf16 gates carry 8 bits: the hardware's exponential and reciprocal are exact enough
+        const float a0 = __fdividef(p.gate_sigmoid ? 1.f : z.x, 1.f + __expf(-fmaxf(z.x, -80.f)));
+        const float a1 = __fdividef(p.gate_sigmoid ? 1.f : z.y, 1.f + __expf(-fmaxf(z.y, -80.f)));
         *reinterpret_cast<__nv_bfloat162*>(o + c) = __floats2bfloat162_rn(acc[i][2 * half] * f * a0, acc[i][2 * half + 1] * f * a1);
       }
     }
@@ -445,6 +530,7 @@ static int launch_retention_output(const RetentionChunkParams& p, int chunks, cu
   const size_t smem = rc_output_smem(p.d, p.e);
   auto kern = retention_chunk_output_kernel<NT>;
   LLMCTL_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
+  LLMCTL_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared));
   kern<<<dim3(chunks, p.nh), 256, smem, s>>>(p);
   return 0;
 }
@@ -527,11 +613,12 @@ LLMCTL_API int llmctl_retention_chunked(const void* q, long long ldq, const void
   if (rot > 0) retention_angles_kernel<<<(tokens * (rot / 2) + 255) / 256, 256, 0, s>>>(positions, freq, rot / 2, (float2*)cs, tokens);
   const size_t smem = rc_sum_smem(d, e);
   LLMCTL_CHECK(cudaFuncSetAttribute(retention_chunk_sum_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
+  LLMCTL_CHECK(cudaFuncSetAttribute(retention_chunk_sum_kernel, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared));
   for (int h0 = 0; h0 < H; h0 += heads_per_pass) {
     p.h0 = h0;
     p.nh = H - h0 < heads_per_pass ? H - h0 : heads_per_pass;
     retention_chunk_sum_kernel<<<dim3(chunks, p.nh), 256, smem, s>>>(p);
-    retention_chunk_chain_kernel<<<dim3(nportions, p.nh, (d * e / 4 + 255) / 256), 256, 0, s>>>(p);
+    retention_chunk_chain_kernel<<<dim3(nportions, p.nh, (d * e / 8 + 255) / 256), 256, 0, s>>>(p);
     const int nt = (e / 8 + 1) / 2;
     const int rc = nt <= 2 ? launch_retention_output<2>(p, chunks, s) : nt <= 4 ? launch_retention_output<4>(p, chunks, s)
                  : nt <= 8 ? launch_retention_output<8>(p, chunks, s) : launch_retention_output<16>(p, chunks, s);

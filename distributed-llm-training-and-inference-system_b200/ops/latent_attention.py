@@ -65,7 +65,7 @@ def rows_per_tile(dtype: torch.dtype, R: int, dr: int, cuda: bool, rows_wanted: 
     (``rows_wanted``: the tokens of a prompt portion, or the heads of a decoding token), else 16."""
     wide = ROWS_PER_TILE_WIDE
     smem = (wide + 64) * (R + dr + 8) * 2 + wide * (68 * 4 + 72 * 2 + 16)
-    ok = cuda and rows_wanted > ROWS_PER_TILE and uses_tensor_cores(dtype, R, dr) and smem <= 227 * 1024
+    ok = cuda and rows_wanted > ROWS_PER_TILE and uses_tensor_cores(dtype, R, dr) and smem <= 225 * 1024
     return wide if ok else ROWS_PER_TILE
 
 
