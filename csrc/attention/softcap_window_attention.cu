@@ -394,9 +394,9 @@ __device__ __forceinline__ float sw_tanh(float x) {
   return 1.f - __fdividef(2.f, 1.f + exp2f(2.f * kSwLog2e * x));
 }
 
-// NT: n-tiles of 8 output columns (e <= 8 NT).  decode = 0: rows of the CTA are the tile's tokens (head blockIdx.y);
+// NT: n-tiles of 8 output columns (e <= 8 NT; FULL: e == 8 NT).  decode = 0: rows of the CTA are the tile's tokens (head blockIdx.y);
 // decode = 1: rows are HB heads of the tile's single token.
-template <int NT, bool SPLIT>
+template <int NT, bool SPLIT, bool FULL>
 __global__ void __launch_bounds__(256, SPLIT ? 1 : 2)
 softcap_attention_mma_kernel(const SoftcapAttnParams p, int decode) {
   extern __shared__ __align__(16) unsigned char sw_smem[];
@@ -489,6 +489,7 @@ softcap_attention_mma_kernel(const SoftcapAttnParams p, int decode) {
   const int warp_first = decode ? p_first : p_first + warp * 16;
   const int warp_last = decode ? p_first : p_first + min(warp * 16 + 15, nvalid - 1);
   const int warp_wb = sw_first_key(warp_first, p);
+  const int warp_wb_last = sw_first_key(warp_last, p);      // rows without a query have position -1: their weights are never stored
   const int qfirst_lo = sw_first_key(max(qpos_lo, 0), p), qfirst_hi = sw_first_key(max(qpos_hi, 0), p);
 
   float O[NT][4];
@@ -532,15 +533,21 @@ softcap_attention_mma_kernel(const SoftcapAttnParams p, int decode) {
       uint32_t ah[4], al[4];
       load_a_frag(ah, Qhi, ldq, warp * 16, ks, lane);
       load_a_frag(al, Qlo, ldq, warp * 16, ks, lane);
-#pragma unroll
-      for (int nt = 0; nt < 4; ++nt) {
-        uint32_t b[2];
-        load_b_frag_nk(b, Kt, ldk, nt * 8, ks, lane);
-        mma_bf16_16816(S[nt], ah, b);
-        mma_bf16_16816(S[nt], al, b);
-      }
+      uint32_t b0[4], b1[4];
+      load_b2_frag_nk(b0, Kt, ldk, 0, ks, lane);
+      load_b2_frag_nk(b1, Kt, ldk, 16, ks, lane);
+      mma_bf16_16816(S[0], ah, b0[0], b0[1]);
+      mma_bf16_16816(S[1], ah, b0[2], b0[3]);
+      mma_bf16_16816(S[2], ah, b1[0], b1[1]);
+      mma_bf16_16816(S[3], ah, b1[2], b1[3]);
+      mma_bf16_16816(S[0], al, b0[0], b0[1]);
+      mma_bf16_16816(S[1], al, b0[2], b0[3]);
+      mma_bf16_16816(S[2], al, b1[0], b1[1]);
+      mma_bf16_16816(S[3], al, b1[2], b1[3]);
     }
     const bool near_tile = warp_first - (k0 + kSwKT - 1) < far;
+    // every key of the tile is visible to every row of the warp: no masks
+    const bool interior = k0 + kSwKT - 1 <= warp_first && k0 + kSwKT <= k_lim && k0 >= warp_wb_last;
     // cap, distance bias, mask; running maximum and sum per row (scores in units of ln 2 from here on)
     float mx_lo = -INFINITY, mx_hi = -INFINITY;
 #pragma unroll
@@ -554,8 +561,10 @@ softcap_attention_mma_kernel(const SoftcapAttnParams p, int decode) {
           s_lo = p.cap * sw_tanh(s_lo / p.cap);
           s_hi = p.cap * sw_tanh(s_hi / p.cap);
         }
-        s_lo -= slope_lo * static_cast<float>(qpos_lo - key);
-        s_hi -= slope_hi * static_cast<float>(qpos_hi - key);
+        if (p.slopes) {
+          s_lo -= slope_lo * static_cast<float>(qpos_lo - key);
+          s_hi -= slope_hi * static_cast<float>(qpos_hi - key);
+        }
         if (tab_lo) {
           if (near_tile) {               // distances outside 0 .. far belong to masked or far keys
             s_lo += tab_lo[min(max(qpos_lo - key, 0), far)];
@@ -567,8 +576,12 @@ softcap_attention_mma_kernel(const SoftcapAttnParams p, int decode) {
         }
         s_lo *= kSwLog2e;
         s_hi *= kSwLog2e;
-        S[nt][j] = (in && sw_visible(qpos_lo, qfirst_lo, key, p.keep_first)) ? s_lo : -INFINITY;
-        S[nt][2 + j] = (in && sw_visible(qpos_hi, qfirst_hi, key, p.keep_first)) ? s_hi : -INFINITY;
+        if (!interior) {
+          if (!in || !sw_visible(qpos_lo, qfirst_lo, key, p.keep_first)) s_lo = -INFINITY;
+          if (!in || !sw_visible(qpos_hi, qfirst_hi, key, p.keep_first)) s_hi = -INFINITY;
+        }
+        S[nt][j] = s_lo;
+        S[nt][2 + j] = s_hi;
         mx_lo = fmaxf(mx_lo, S[nt][j]);
         mx_hi = fmaxf(mx_hi, S[nt][2 + j]);
       }
@@ -606,12 +619,14 @@ softcap_attention_mma_kernel(const SoftcapAttnParams p, int decode) {
       sw_split_pack(S[2 * kk + 1][0], S[2 * kk + 1][1], ph[2], pl[2]);
       sw_split_pack(S[2 * kk + 1][2], S[2 * kk + 1][3], ph[3], pl[3]);
 #pragma unroll
-      for (int nt = 0; nt < NT; ++nt) {
-        if (nt * 8 < e) {
-          uint32_t b[2];
-          load_b_frag_kn(b, Vt, ldv, kk * 16, nt * 8, lane);
-          mma_bf16_16816(O[nt], ph, b);
-          mma_bf16_16816(O[nt], pl, b);
+      for (int nt = 0; nt < NT; nt += 2) {
+        if (FULL || nt * 8 < e) {          // columns past e come from the rows' padding and are never stored
+          uint32_t b[4];
+          load_b2_frag_kn(b, Vt, ldv, kk * 16, nt * 8, lane);
+          mma_bf16_16816(O[nt], ph, b[0], b[1]);
+          mma_bf16_16816(O[nt + 1], ph, b[2], b[3]);
+          mma_bf16_16816(O[nt], pl, b[0], b[1]);
+          mma_bf16_16816(O[nt + 1], pl, b[2], b[3]);
         }
       }
     }
@@ -716,7 +731,7 @@ static int launch_softcap_attention_mma(const SoftcapAttnParams& p, int ntiles, 
   const dim3 grid(ntiles * p.splits, decode ? p.H / p.HB : p.H);
 #define LLMCTL_SW_LAUNCH(NT)                                                                                                     \
   do {                                                                                                                           \
-    auto kern = softcap_attention_mma_kernel<NT, SPLIT>;                                                                         \
+    auto kern = p.e == 8 * NT ? softcap_attention_mma_kernel<NT, SPLIT, true> : softcap_attention_mma_kernel<NT, SPLIT, false>;  \
     if (smem > 46 * 1024) LLMCTL_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem))); \
     kern<<<grid, warps * 32, smem, s>>>(p, decode);                                                                              \
   } while (0)

@@ -42,6 +42,27 @@ __device__ __forceinline__ void load_b_frag_kn(uint32_t (&b)[2], const __nv_bflo
   asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];\n" : "=r"(b[0]), "=r"(b[1]) : "r"(addr));
 }
 
+// Two neighbouring B fragments (n0 .. n0 + 7 in b[0], b[1]; n0 + 8 .. n0 + 15 in b[2], b[3]) by one ldmatrix.x4: operand stored
+// [n][k] / [k][n] row-major (same alignment rules).
+__device__ __forceinline__ void load_b2_frag_nk(uint32_t (&b)[4], const __nv_bfloat16* m, int ld, int n0, int k0, int lane) {
+  const __nv_bfloat16* p = m + (n0 + (lane & 7) + ((lane >> 4) << 3)) * ld + k0 + (((lane >> 3) & 1) << 3);
+  const uint32_t addr = static_cast<uint32_t>(__cvta_generic_to_shared(p));
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n"
+               : "=r"(b[0]), "=r"(b[1]), "=r"(b[2]), "=r"(b[3])
+               : "r"(addr));
+}
+__device__ __forceinline__ void load_b2_frag_kn(uint32_t (&b)[4], const __nv_bfloat16* m, int ld, int k0, int n0, int lane) {
+  const __nv_bfloat16* p = m + (k0 + (lane & 15)) * ld + n0 + ((lane >> 4) << 3);
+  const uint32_t addr = static_cast<uint32_t>(__cvta_generic_to_shared(p));
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];\n"
+               : "=r"(b[0]), "=r"(b[1]), "=r"(b[2]), "=r"(b[3])
+               : "r"(addr));
+}
+__device__ __forceinline__ void mma_bf16_16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  const uint32_t b[2] = {b0, b1};
+  mma_bf16_16816(c, a, b);
+}
+
 // 16-byte asynchronous global -> shared copies (both addresses 16-byte aligned), grouped and awaited per thread.
 __device__ __forceinline__ void cp_async_16(void* smem, const void* gmem) {
   const uint32_t s = static_cast<uint32_t>(__cvta_generic_to_shared(smem));

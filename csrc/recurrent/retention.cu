@@ -208,22 +208,6 @@ __device__ __forceinline__ void rc_load_rows(const __nv_bfloat16* x, long long l
   }
 }
 
-// two neighbouring B fragments (8 columns each) by one ldmatrix: operand stored [n][k] / [k][n]
-__device__ __forceinline__ void rc_b2_nk(uint32_t (&b)[4], const __nv_bfloat16* m, int ld, int n0, int k0, int lane) {
-  const __nv_bfloat16* p = m + (n0 + (lane & 7) + ((lane >> 4) << 3)) * ld + k0 + (((lane >> 3) & 1) << 3);
-  const uint32_t addr = static_cast<uint32_t>(__cvta_generic_to_shared(p));
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n" : "=r"(b[0]), "=r"(b[1]), "=r"(b[2]), "=r"(b[3]) : "r"(addr));
-}
-__device__ __forceinline__ void rc_b2_kn(uint32_t (&b)[4], const __nv_bfloat16* m, int ld, int k0, int n0, int lane) {
-  const __nv_bfloat16* p = m + (k0 + (lane & 15)) * ld + n0 + ((lane >> 4) << 3);
-  const uint32_t addr = static_cast<uint32_t>(__cvta_generic_to_shared(p));
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];\n" : "=r"(b[0]), "=r"(b[1]), "=r"(b[2]), "=r"(b[3]) : "r"(addr));
-}
-__device__ __forceinline__ void rc_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  const uint32_t b[2] = {b0, b1};
-  mma_bf16_16816(c, a, b);
-}
-
 // A fragment of A[m][k] = s[k0 + k][m0 + m] (operand stored [k][m] row-major): ldmatrix with transposition
 __device__ __forceinline__ void rc_a_frag_km(uint32_t (&a)[4], const __nv_bfloat16* s, int ld, int m0, int k0, int lane) {
   const __nv_bfloat16* p = s + (k0 + (lane & 7) + ((lane >> 4) << 3)) * ld + m0 + (((lane >> 3) & 1) << 3);
@@ -265,11 +249,11 @@ retention_chunk_sum_kernel(const RetentionChunkParams p) {
       for (int i = 0; i < 4; i += 2)
         if (n0 + 8 * i < e) {                          // e is a multiple of 16
           uint32_t bf[4];
-          rc_b2_kn(bf, V, ldv, ks * 16, n0 + 8 * i, lane);
-          rc_mma(acc[i], ah, bf[0], bf[1]);
-          rc_mma(acc[i + 1], ah, bf[2], bf[3]);
-          rc_mma(acc[i], al, bf[0], bf[1]);
-          rc_mma(acc[i + 1], al, bf[2], bf[3]);
+          load_b2_frag_kn(bf, V, ldv, ks * 16, n0 + 8 * i, lane);
+          mma_bf16_16816(acc[i], ah, bf[0], bf[1]);
+          mma_bf16_16816(acc[i + 1], ah, bf[2], bf[3]);
+          mma_bf16_16816(acc[i], al, bf[0], bf[1]);
+          mma_bf16_16816(acc[i + 1], al, bf[2], bf[3]);
         }
     }
 #pragma unroll
@@ -371,14 +355,14 @@ retention_chunk_output_kernel(const RetentionChunkParams p) {
       for (int i = 0; i < 8; i += 2)
         if (i < 2 * (rg + 1)) {                        // later keys are masked for all rows of the warp
           uint32_t bh[4], bl[4];
-          rc_b2_nk(bh, Kh, ldq, 8 * i, ks, lane);
-          rc_b2_nk(bl, Kl, ldq, 8 * i, ks, lane);
-          rc_mma(s[i], ah, bh[0], bh[1]);
-          rc_mma(s[i + 1], ah, bh[2], bh[3]);
-          rc_mma(s[i], al, bh[0], bh[1]);
-          rc_mma(s[i + 1], al, bh[2], bh[3]);
-          rc_mma(s[i], ah, bl[0], bl[1]);
-          rc_mma(s[i + 1], ah, bl[2], bl[3]);
+          load_b2_frag_nk(bh, Kh, ldq, 8 * i, ks, lane);
+          load_b2_frag_nk(bl, Kl, ldq, 8 * i, ks, lane);
+          mma_bf16_16816(s[i], ah, bh[0], bh[1]);
+          mma_bf16_16816(s[i + 1], ah, bh[2], bh[3]);
+          mma_bf16_16816(s[i], al, bh[0], bh[1]);
+          mma_bf16_16816(s[i + 1], al, bh[2], bh[3]);
+          mma_bf16_16816(s[i], ah, bl[0], bl[1]);
+          mma_bf16_16816(s[i + 1], ah, bl[2], bl[3]);
         }
     }
 #pragma unroll
@@ -443,14 +427,14 @@ retention_chunk_output_kernel(const RetentionChunkParams p) {
           for (int i = 0; i < NT; i += 2)
             if (n_base + 8 * i < e) {
               uint32_t bh[4], bl[4];
-              rc_b2_kn(bh, Sh, ldv, ks, n_base + 8 * i, lane);
-              rc_b2_kn(bl, Sl, ldv, ks, n_base + 8 * i, lane);
-              rc_mma(acc[i], ah, bh[0], bh[1]);
-              rc_mma(acc[i + 1], ah, bh[2], bh[3]);
-              rc_mma(acc[i], al, bh[0], bh[1]);
-              rc_mma(acc[i + 1], al, bh[2], bh[3]);
-              rc_mma(acc[i], ah, bl[0], bl[1]);
-              rc_mma(acc[i + 1], ah, bl[2], bl[3]);
+              load_b2_frag_kn(bh, Sh, ldv, ks, n_base + 8 * i, lane);
+              load_b2_frag_kn(bl, Sl, ldv, ks, n_base + 8 * i, lane);
+              mma_bf16_16816(acc[i], ah, bh[0], bh[1]);
+              mma_bf16_16816(acc[i + 1], ah, bh[2], bh[3]);
+              mma_bf16_16816(acc[i], al, bh[0], bh[1]);
+              mma_bf16_16816(acc[i + 1], al, bh[2], bh[3]);
+              mma_bf16_16816(acc[i], ah, bl[0], bl[1]);
+              mma_bf16_16816(acc[i + 1], ah, bl[2], bl[3]);
             }
         }
       }
@@ -475,11 +459,11 @@ retention_chunk_output_kernel(const RetentionChunkParams p) {
         for (int i = 0; i < NT; i += 2)
           if (n_base + 8 * i < e) {
             uint32_t b[4];
-            rc_b2_kn(b, V, ldv, kk * 16, n_base + 8 * i, lane);
-            rc_mma(acc[i], ph[kk], b[0], b[1]);
-            rc_mma(acc[i + 1], ph[kk], b[2], b[3]);
-            rc_mma(acc[i], pl[kk], b[0], b[1]);
-            rc_mma(acc[i + 1], pl[kk], b[2], b[3]);
+            load_b2_frag_kn(b, V, ldv, kk * 16, n_base + 8 * i, lane);
+            mma_bf16_16816(acc[i], ph[kk], b[0], b[1]);
+            mma_bf16_16816(acc[i + 1], ph[kk], b[2], b[3]);
+            mma_bf16_16816(acc[i], pl[kk], b[0], b[1]);
+            mma_bf16_16816(acc[i + 1], pl[kk], b[2], b[3]);
           }
       }
     float s_lo = 0.f, s_hi = 0.f;

@@ -159,7 +159,7 @@ def softcap_window_attention(q: torch.Tensor, cache: torch.Tensor, block_tables:
         elif not splits:
             seen = min(max_context, window + keep_first) if window > 0 else max_context
             seen = min(seen, chunk + keep_first) if chunk > 0 else seen
-            splits = key_splits(n * (H // hb), seen, 8 if mma else 2, 64 if mma else 128)
+            splits = key_splits(n * (H // hb), seen, 8 if mma else 2, 128)
         part_ml = torch.empty(n * (H // hb) * splits * 64, dtype=torch.float32, device=q.device) if splits > 1 else None
         part_o = torch.empty(n * (H // hb) * splits * 32 * e, dtype=torch.float32, device=q.device) if splits > 1 else None
         native.call("llmctl_softcap_window_attention", q.data_ptr(), cache.data_ptr(), block_tables.data_ptr(), block_tables.shape[1],

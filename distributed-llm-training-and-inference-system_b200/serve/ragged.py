@@ -117,9 +117,10 @@ class RaggedBatch:
                     out_rows[o] = t + w
                     o += 1
                 for k, width in enumerate(self._tile_tokens):
-                    for s in range(0, n, width):
-                        tiles[k][ti[k]] = (t + s, min(width, n - s), b, 0)
-                        ti[k] += 1
+                    first = np.arange(0, n, width)
+                    rows = tiles[k][ti[k]:ti[k] + len(first)]
+                    rows[:, 0], rows[:, 1], rows[:, 2], rows[:, 3] = t + first, np.minimum(width, n - first), b, 0
+                    ti[k] += len(first)
             t += n
         if self._dev is not self._host:
             self._dev.copy_(self._host, non_blocking=True)
