@@ -89,6 +89,8 @@ retention_prepare_kernel(const RetentionPrepParams p) {
 // chunks of 64 tokens on the tensor cores
 // ---------------------------------------------------------------------------------------------------------------
 constexpr int kRcTokens = 64;
+constexpr int kRcEarly = 2;         // stages of 16 state rows that the output kernel fills before it has read the keys
+constexpr int kRcFlight = 6;        // most slices of the state in flight
 
 struct RetentionChunkParams {
   const __nv_bfloat16* q;     // [T, H d] (row strides below)
@@ -131,29 +133,33 @@ __device__ __forceinline__ void rc_split4(const float (&v)[4], uint2& hi, uint2&
   lo = make_uint2(pack_bf16x2(r[0], r[1]), pack_bf16x2(r[2], r[3]));
 }
 
-// Rows j of a chunk (x + j ld, d numbers): rotated, times factor [* decay^(last - j)], split into hi and lo
-// [64][d + 8] in shared memory; rows past n are zeros.  An item is four pairs or four unrotated numbers; the loads of IT items per
-// thread are in flight together.
-template <int IT, bool DECAY>
-__device__ __forceinline__ void rc_load_rotated(const __nv_bfloat16* x, long long ld, const float2* cs, int half, int d, int n, float factor,
-                                                float log2_decay, int last, __nv_bfloat16* hi, __nv_bfloat16* lo) {
+// Rows j of a chunk (x[m] + j ld[m], d numbers each, NM operands): rotated, times factor[m] [* decay^(last - j)], split into hi and lo
+// [64][d + 8] in shared memory; rows past n are zeros.  An item is four pairs or four unrotated numbers of every operand; the
+// loads of IT items per thread are in flight together.
+template <int NM, int IT, bool DECAY>
+__device__ __forceinline__ void rc_load_rotated(const __nv_bfloat16* const (&x)[NM], const long long (&ld)[NM], const float2* cs, int half, int d, int n,
+                                                const float (&factor)[NM], float log2_decay, int last, __nv_bfloat16* const (&hi)[NM],
+                                                __nv_bfloat16* const (&lo)[NM]) {
   const int pairs = half >> 2, per = (d >> 2) - pairs, lds = d + 8, total = kRcTokens * per;
   const int dj = 256 / per, dk = 256 - dj * per;       // CTAs of 256 threads
   int i = threadIdx.x, j = i / per, k = i - j * per;
   while (i < total) {
-    float a[IT][4], b[IT][4], w[IT][8];
+    uint2 a[IT][NM], b[IT][NM];
+    float w[IT][8];
     int jj[IT], cc[IT];
 #pragma unroll
     for (int u = 0; u < IT; ++u) {
       jj[u] = i < total ? j : -1;
       cc[u] = k < pairs ? k << 2 : (k << 2) + half;
 #pragma unroll
-      for (int v = 0; v < 4; ++v) a[u][v] = b[u][v] = 0.f;
+      for (int m = 0; m < NM; ++m) a[u][m] = b[u][m] = make_uint2(0u, 0u);
       if (i < total && j < n) {
-        load_vec<4>(x + j * ld + cc[u], a[u]);
+#pragma unroll
+        for (int m = 0; m < NM; ++m) a[u][m] = *reinterpret_cast<const uint2*>(x[m] + j * ld[m] + cc[u]);
         if (cc[u] < half) {
-          load_vec<4>(x + j * ld + cc[u] + half, b[u]);
-          const float* t = reinterpret_cast<const float*>(cs + static_cast<long long>(j) * half + cc[u]);
+#pragma unroll
+          for (int m = 0; m < NM; ++m) b[u][m] = *reinterpret_cast<const uint2*>(x[m] + j * ld[m] + cc[u] + half);
+          const float* t = reinterpret_cast<const float*>(cs + j * half + cc[u]);
           *reinterpret_cast<float4*>(w[u]) = *reinterpret_cast<const float4*>(t);
           *reinterpret_cast<float4*>(w[u] + 4) = *reinterpret_cast<const float4*>(t + 4);
         }
@@ -167,27 +173,36 @@ __device__ __forceinline__ void rc_load_rotated(const __nv_bfloat16* x, long lon
     for (int u = 0; u < IT; ++u) {
       const int row = jj[u], c = cc[u];
       if (row < 0) continue;
-      float f = factor;
-      if (DECAY) f = row < n ? factor * rc_power(log2_decay, last - row) : 0.f;
-      if (c < half && row < n) {
+      float pw = 1.f;
+      if (DECAY) pw = row < n ? rc_power(log2_decay, last - row) : 0.f;
+      const int at = row * lds + c;
 #pragma unroll
-        for (int v = 0; v < 4; ++v) {
-          const float p = a[u][v], q = b[u][v];
-          a[u][v] = (p * w[u][2 * v] - q * w[u][2 * v + 1]) * f;
-          b[u][v] = (q * w[u][2 * v] + p * w[u][2 * v + 1]) * f;
+      for (int m = 0; m < NM; ++m) {
+        const float f = factor[m] * pw;
+        float p[4] = {__uint_as_float(a[u][m].x << 16), __uint_as_float(a[u][m].x & 0xffff0000u), __uint_as_float(a[u][m].y << 16),
+                      __uint_as_float(a[u][m].y & 0xffff0000u)};
+        uint2 h, l;
+        if (c < half) {
+          float q[4] = {__uint_as_float(b[u][m].x << 16), __uint_as_float(b[u][m].x & 0xffff0000u), __uint_as_float(b[u][m].y << 16),
+                        __uint_as_float(b[u][m].y & 0xffff0000u)};
+          if (row < n) {
+#pragma unroll
+            for (int v = 0; v < 4; ++v) {
+              const float p0 = p[v], q0 = q[v];
+              p[v] = (p0 * w[u][2 * v] - q0 * w[u][2 * v + 1]) * f;
+              q[v] = (q0 * w[u][2 * v] + p0 * w[u][2 * v + 1]) * f;
+            }
+          }
+          rc_split4(q, h, l);
+          *reinterpret_cast<uint2*>(hi[m] + at + half) = h;
+          *reinterpret_cast<uint2*>(lo[m] + at + half) = l;
+        } else {
+#pragma unroll
+          for (int v = 0; v < 4; ++v) p[v] *= f;
         }
-      } else {
-#pragma unroll
-        for (int v = 0; v < 4; ++v) a[u][v] *= f;
-      }
-      uint2 h, l;
-      rc_split4(a[u], h, l);
-      *reinterpret_cast<uint2*>(hi + row * lds + c) = h;
-      *reinterpret_cast<uint2*>(lo + row * lds + c) = l;
-      if (c < half) {
-        rc_split4(b[u], h, l);
-        *reinterpret_cast<uint2*>(hi + row * lds + c + half) = h;
-        *reinterpret_cast<uint2*>(lo + row * lds + c + half) = l;
+        rc_split4(p, h, l);
+        *reinterpret_cast<uint2*>(hi[m] + at) = h;
+        *reinterpret_cast<uint2*>(lo[m] + at) = l;
       }
     }
   }
@@ -232,7 +247,8 @@ retention_chunk_sum_kernel(const RetentionChunkParams p) {
   const float lg = rc_log2_decay(p.dm[h]);
   rc_load_rows(p.v + t0 * p.ldv + h * e, p.ldv, e, n, V, ldv);
   cp_async_commit();
-  rc_load_rotated<2, true>(p.k + t0 * p.ldk + h * d, p.ldk, p.cs + t0 * p.half, p.half, d, n, 1.f / sqrtf(static_cast<float>(d)), lg, n - 1, Kh, Kl);
+  rc_load_rotated<1, 4, true>({p.k + t0 * p.ldk + h * d}, {p.ldk}, p.cs + t0 * p.half, p.half, d, n, {1.f / sqrtf(static_cast<float>(d))}, lg, n - 1,
+                              {Kh}, {Kl});
   cp_async_wait_all();
   __syncthreads();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3;
@@ -310,8 +326,8 @@ retention_chunk_chain_kernel(const RetentionChunkParams p) {
   if (st) store8_f32(st, S);
 }
 
-// Outputs of a chunk and head.  Warp (r, c) = (warp % 4, warp / 4) owns 16 tokens and half of the value columns (NT tiles of 8).
-template <int NT>
+// Outputs of a chunk and head (FULL: e == 16 NT).  Warp (r, c) = (warp % 4, warp / 4) owns 16 tokens and half of the value columns (NT tiles of 8).
+template <int NT, bool FULL>
 __global__ void __launch_bounds__(256, NT <= 8 ? 2 : 1)
 retention_chunk_output_kernel(const RetentionChunkParams p) {
   extern __shared__ __align__(16) unsigned char rc_smem[];
@@ -326,16 +342,36 @@ retention_chunk_output_kernel(const RetentionChunkParams p) {
   __nv_bfloat16* Qh = reinterpret_cast<__nv_bfloat16*>(rc_smem);
   __nv_bfloat16* Ql = Qh + kRcTokens * ldq;
   __nv_bfloat16* V = Ql + kRcTokens * ldq;
-  __nv_bfloat16* Kh = V + kRcTokens * ldv;             // keys, then two stages of 32 rows of the state (hi, lo)
+  __nv_bfloat16* ring = V + kRcTokens * ldv;           // stages of 16 state rows (hi, lo): kRcEarly of them for their own ...
+  __nv_bfloat16* Kh = ring + kRcEarly * 32 * ldv;      // ... and the keys' place, which holds as many more afterwards as fit
   __nv_bfloat16* Kl = Kh + kRcTokens * ldq;
   const float2* cs = p.cs + t0 * p.half;
   const float lg = rc_log2_decay(p.dm[h]);
+  const int slices = has_state ? d / 16 : 0, stages = kRcEarly + 128 * ldq / (32 * ldv);
+  const int per = e >> 3, dr = 256 / per, dk = 256 - dr * per, first_r = threadIdx.x / per, first_k = threadIdx.x - first_r * per;
+  const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(p.scratch + (static_cast<long long>(blockIdx.x) * p.nh + blockIdx.y) * d * e);
+  auto fetch = [&](int sl) {                           // rows 16 sl .. of the state; 8 hi and 8 lo numbers lie next to each other
+    __nv_bfloat16* Sh = ring + (sl % stages) * 32 * ldv;
+    for (int r = first_r, k = first_k; r < 16; r += dr, k += dk) {
+      if (k >= per) {
+        k -= per;
+        if (++r >= 16) break;
+      }
+      const int c = k << 3;
+      const __nv_bfloat16* u = src + ((sl * 16 + r) * e + c) * 2;
+      cp_async_16(Sh + r * ldv + c, u);
+      cp_async_16(Sh + (16 + r) * ldv + c, u + 8);
+    }
+  };
   if (threadIdx.x <= kRcTokens) power[threadIdx.x] = rc_power(lg, threadIdx.x);
   rc_load_rows(p.v + t0 * p.ldv + h * e, p.ldv, e, n, V, ldv);
   cp_async_commit();
-  rc_load_rotated<4, false>(p.q + t0 * p.ldq + h * d, p.ldq, cs, p.half, d, n, 1.f, 0.f, 0, Qh, Ql);
-  rc_load_rotated<4, false>(p.k + t0 * p.ldk + h * d, p.ldk, cs, p.half, d, n, 1.f / sqrtf(static_cast<float>(d)), 0.f, 0, Kh, Kl);
-  cp_async_wait_all();
+  for (int sl = 0; sl < kRcEarly; ++sl) {              // one group per slice from here on, empty past the last one
+    if (sl < slices) fetch(sl);
+    cp_async_commit();
+  }
+  rc_load_rotated<2, 4, false>({p.q + t0 * p.ldq + h * d, p.k + t0 * p.ldk + h * d}, {p.ldq, p.ldk}, cs, p.half, d, n,
+                               {1.f, 1.f / sqrtf(static_cast<float>(d))}, 0.f, 0, {Qh, Kh}, {Ql, Kl});
   __syncthreads();
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
   const int rg = warp & 3, r0 = rg * 16, n_base = (warp >> 2) * NT * 8;
@@ -388,61 +424,40 @@ retention_chunk_output_kernel(const RetentionChunkParams p) {
 #pragma unroll
     for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
   if (has_state) {                                     // uniform over the CTA
-    constexpr int SR = kRcTokens / 2;                  // state rows per stage
-    const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(p.scratch + (static_cast<long long>(blockIdx.x) * p.nh + blockIdx.y) * d * e);
-    const int per = e >> 3, slices = (d + SR - 1) / SR;
-    const int dr = 256 / per, dk = 256 - dr * per, first_r = tid / per, first_k = tid - first_r * per;
-    auto fetch = [&](int sl) {                         // rows sl SR .. of the state; 8 hi and 8 lo numbers lie next to each other
-      __nv_bfloat16* Sh = Kh + (sl & 1) * 2 * SR * ldv;
-      const int rows = min(SR, d - sl * SR);
-      int r = first_r, k = first_k;
-      for (; r < rows; r += dr, k += dk) {
-        if (k >= per) {
-          k -= per;
-          if (++r >= rows) break;
-        }
-        const int c = k << 3;
-        const __nv_bfloat16* u = src + (static_cast<long long>(sl * SR + r) * e + c) * 2;
-        cp_async_16(Sh + r * ldv + c, u);
-        cp_async_16(Sh + (SR + r) * ldv + c, u + 8);
-      }
-    };
     __syncthreads();                                   // the readers of the keys are done
-    fetch(0);
-    cp_async_commit();
-    if (slices > 1) fetch(1);
-    cp_async_commit();
-    for (int sl = 0; sl < slices; ++sl) {
-      cp_async_wait_prior();
-      __syncthreads();                                 // slice sl has landed
-      const __nv_bfloat16* Sh = Kh + (sl & 1) * 2 * SR * ldv;
-      const __nv_bfloat16* Sl = Sh + SR * ldv;
-      const int rows = min(SR, d - sl * SR);
-      if (active) {
-        for (int ks = 0; ks < rows; ks += 16) {
-          uint32_t ah[4], al[4];
-          load_a_frag(ah, Qh, ldq, r0, sl * SR + ks, lane);
-          load_a_frag(al, Ql, ldq, r0, sl * SR + ks, lane);
-#pragma unroll
-          for (int i = 0; i < NT; i += 2)
-            if (n_base + 8 * i < e) {
-              uint32_t bh[4], bl[4];
-              load_b2_frag_kn(bh, Sh, ldv, ks, n_base + 8 * i, lane);
-              load_b2_frag_kn(bl, Sl, ldv, ks, n_base + 8 * i, lane);
-              mma_bf16_16816(acc[i], ah, bh[0], bh[1]);
-              mma_bf16_16816(acc[i + 1], ah, bh[2], bh[3]);
-              mma_bf16_16816(acc[i], al, bh[0], bh[1]);
-              mma_bf16_16816(acc[i + 1], al, bh[2], bh[3]);
-              mma_bf16_16816(acc[i], ah, bl[0], bl[1]);
-              mma_bf16_16816(acc[i + 1], ah, bl[2], bl[3]);
-            }
-        }
-      }
-      if (sl + 2 < slices) {
-        __syncthreads();                               // its readers are done: the stage may be overwritten
-        fetch(sl + 2);
-      }
+    for (int sl = kRcEarly; sl < kRcFlight; ++sl) {    // kRcFlight groups in flight
+      if (sl < slices && sl < stages) fetch(sl);
       cp_async_commit();
+    }
+    const int ahead = min(stages, kRcFlight);          // slices asked for so far
+    for (int sl = 0; sl < slices; ++sl) {
+      // slice s >= ahead is in group kRcFlight + s + 1 - ahead: at most kRcFlight - 2 younger groups may be pending, none with a short ring
+      if (ahead == kRcFlight) asm volatile("cp.async.wait_group %0;\n" ::"n"(kRcFlight - 2) : "memory");
+      else cp_async_wait_all();
+      __syncthreads();                                 // slice sl has landed, everyone is done with slice sl - 1
+      const int next = sl - 1 + ahead;                 // goes where slice sl - 1 (or nothing yet) was
+      if (sl > 0 && next < slices) fetch(next);
+      cp_async_commit();
+      if (active) {
+        const __nv_bfloat16* Sh = ring + (sl % stages) * 32 * ldv;
+        const __nv_bfloat16* Sl = Sh + 16 * ldv;
+        uint32_t ah[4], al[4];
+        load_a_frag(ah, Qh, ldq, r0, sl * 16, lane);
+        load_a_frag(al, Ql, ldq, r0, sl * 16, lane);
+#pragma unroll
+        for (int i = 0; i < NT; i += 2)
+          if (FULL || n_base + 8 * i < e) {
+            uint32_t bh[4], bl[4];
+            load_b2_frag_kn(bh, Sh, ldv, 0, n_base + 8 * i, lane);
+            load_b2_frag_kn(bl, Sl, ldv, 0, n_base + 8 * i, lane);
+            mma_bf16_16816(acc[i], ah, bh[0], bh[1]);
+            mma_bf16_16816(acc[i + 1], ah, bh[2], bh[3]);
+            mma_bf16_16816(acc[i], al, bh[0], bh[1]);
+            mma_bf16_16816(acc[i + 1], al, bh[2], bh[3]);
+            mma_bf16_16816(acc[i], ah, bl[0], bl[1]);
+            mma_bf16_16816(acc[i + 1], ah, bl[2], bl[3]);
+          }
+      }
     }
     const float f_lo = power[r0 + g + 1], f_hi = power[r0 + g + 9];
 #pragma unroll
@@ -451,13 +466,26 @@ retention_chunk_output_kernel(const RetentionChunkParams p) {
       acc[i][2] *= f_hi, acc[i][3] *= f_hi;
     }
   }
+  uint32_t gz[2][NT];                                  // gates, asked for before the last products
+#pragma unroll
+  for (int half = 0; half < 2; ++half) {
+    const int r = r0 + g + 8 * half;
+    const __nv_bfloat16* gr = p.gate + (t0 + min(r, n - 1)) * p.ldg + h * e + n_base + 2 * t;
+#pragma unroll
+    for (int i = 0; i < NT; ++i)
+      if (FULL || n_base + 8 * i < e) gz[half][i] = *reinterpret_cast<const uint32_t*>(gr + 8 * i);
+  }
+  if (!has_state) {                                    // the values' copies may still be in flight
+    cp_async_wait_all();
+    __syncthreads();
+  }
   if (active) {
 #pragma unroll
     for (int kk = 0; kk < 4; ++kk)
       if (kk <= rg) {
 #pragma unroll
         for (int i = 0; i < NT; i += 2)
-          if (n_base + 8 * i < e) {
+          if (FULL || n_base + 8 * i < e) {
             uint32_t b[4];
             load_b2_frag_kn(b, V, ldv, kk * 16, n_base + 8 * i, lane);
             mma_bf16_16816(acc[i], ph[kk], b[0], b[1]);
@@ -488,13 +516,12 @@ retention_chunk_output_kernel(const RetentionChunkParams p) {
     if (r >= n) continue;
     const float f = 1.f / sqrtf((row_ss[0][r] + row_ss[1][r]) / static_cast<float>(e) + p.eps);
     const long long tok = t0 + r;
-    const __nv_bfloat16* gr = p.gate + tok * p.ldg + h * e;
     __nv_bfloat16* o = p.out + (tok * p.H + h) * e;
 #pragma unroll
     for (int i = 0; i < NT; ++i) {
       const int c = n_base + 8 * i + 2 * t;
-      if (n_base + 8 * i < e) {
-        const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gr + c));
+      if (FULL || n_base + 8 * i < e) {
+        const float2 z = make_float2(__uint_as_float(gz[half][i] << 16), __uint_as_float(gz[half][i] & 0xffff0000u));
         // bf16 gates carry 8 bits: the hardware's exponential and reciprocal are exact enough
         const float a0 = __fdividef(p.gate_sigmoid ? 1.f : z.x, 1.f + __expf(-fmaxf(z.x, -80.f)));
         const float a1 = __fdividef(p.gate_sigmoid ? 1.f : z.y, 1.f + __expf(-fmaxf(z.y, -80.f)));
@@ -506,13 +533,13 @@ retention_chunk_output_kernel(const RetentionChunkParams p) {
 
 static size_t rc_sum_smem(int d, int e) { return sizeof(__nv_bfloat16) * kRcTokens * (2 * static_cast<size_t>(d + 8) + (e + 8)); }
 static size_t rc_output_smem(int d, int e) {
-  return sizeof(__nv_bfloat16) * kRcTokens * (2 * static_cast<size_t>(d + 8) + (e + 8) + 2 * static_cast<size_t>((d > e ? d : e) + 8));
+  return sizeof(__nv_bfloat16) * (kRcTokens * (4 * static_cast<size_t>(d + 8) + (e + 8)) + kRcEarly * 32 * static_cast<size_t>(e + 8));
 }
 
 template <int NT>
 static int launch_retention_output(const RetentionChunkParams& p, int chunks, cudaStream_t s) {
   const size_t smem = rc_output_smem(p.d, p.e);
-  auto kern = retention_chunk_output_kernel<NT>;
+  auto kern = p.e == 16 * NT ? retention_chunk_output_kernel<NT, true> : retention_chunk_output_kernel<NT, false>;
   LLMCTL_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
   LLMCTL_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared));
   kern<<<dim3(chunks, p.nh), 256, smem, s>>>(p);

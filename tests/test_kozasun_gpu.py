@@ -195,7 +195,8 @@ def portions_of(lens, pos, slots, device="cpu"):
 
 # sizes on every padded row count and beside it, odd and vector-aligned value sizes, several column blocks
 @pytest.mark.parametrize("H,d,e,rot", [(4, 6, 10, 4), (2, 32, 32, 32), (3, 40, 36, 20), (4, 64, 100, 64), (2, 128, 128, 128), (3, 97, 33, 0), (2, 256, 64, 64),
-                                       (1, 1, 1, 0), (2, 128, 256, 64), (2, 64, 128, 32), (5, 48, 80, 16)])
+                                       (1, 1, 1, 0), (2, 128, 256, 64), (2, 64, 128, 32), (5, 48, 80, 16),
+                                       (2, 16, 256, 8), (1, 112, 224, 104)])
 def test_retention_kernels(cuda_device, H, d, e, rot):
     """Prompts of unequal lengths side by side (one without a slot, one at position 0 over garbage), then decoding steps by the
     single-launch kernel, all from the same evolving states."""
@@ -210,7 +211,7 @@ def test_retention_kernels(cuda_device, H, d, e, rot):
         st = torch.randn(4, H, d, e)
         sg = st.clone().to(dev)
         pos, slots = [5, 0, 9], [2, 0, -1]
-        for lens in ([19, 137, 3], [2, 1, 16], [1, 1, 1], [1, 1, 1], [73, 1, 2], [1, 1, 1], [64, 65, 63]):
+        for lens in ([19, 137, 3], [2, 1, 16], [1, 1, 1], [1, 1, 1], [73, 1, 2], [1, 1, 1], [64, 65, 63], [2, 330, 128]):
             p = torch.randn(sum(lens), 2 * nk + 2 * nv + (8 if (nk + nv) % 8 == 0 else 3)).to(dt)
             po, ps = portions_of(lens, pos, slots)
 
